@@ -70,7 +70,8 @@ extern "C" int qv_bias_attn_prepare(void* q_out, int ld_qo, const float* proj, i
 }
 
 // Queries and keys that are rotated and then unit-normed, values that may be blended with another layer's:
-//   q, k heads: the first `rot` entries rotated in split halves (entry i with entry i + rot/2, angles of row tok_pos of cos_sin),
+//   q, k heads: the first `rot` entries rotated in split halves (entry i with entry i + rot/2, angles of row tok_pos of cos_sin)
+//   or, with `interleaved`, in neighbouring pairs (entry 2i with entry 2i + 1),
 //   then, if `unit`, divided by the root mean square over the head (eps under the root); q also times head_temp[h] (or 1);
 //   v = (1 - lam) v + lam v_first[t] where v_first is given (float32 [T, G * dv], row stride ld_vf).
 // proj [T, ...] float32 with [q | k | v] at q_off, k_off, v_off; q -> q_out (compute type), k and v -> the token's cache row
@@ -78,7 +79,7 @@ extern "C" int qv_bias_attn_prepare(void* q_out, int ld_qo, const float* proj, i
 template <typename T>
 __global__ void __launch_bounds__(256) rot_norm_prepare_kernel(T* __restrict__ q_out, int ld_qo, const float* __restrict__ proj, int ld_p,
                                                               int q_off, int k_off, int v_off, T* __restrict__ cache,
-                                                              const float2* __restrict__ cos_sin, int table_rows, int rot, int unit,
+                                                              const float2* __restrict__ cos_sin, int table_rows, int rot, int interleaved, int unit,
                                                               float eps, const float* __restrict__ head_temp,
                                                               const float* __restrict__ v_first, int ld_vf, float lam,
                                                               const int* __restrict__ tok_pos, const int* __restrict__ tok_seg,
@@ -102,10 +103,11 @@ __global__ void __launch_bounds__(256) rot_norm_prepare_kernel(T* __restrict__ q
     for (int i = lane; i < n; i += 32) x[i] = src[i];
     __syncwarp();
     for (int i = lane; i < half; i += 32) {
-      const float a = x[i], b = x[i + half];
+      const int iu = interleaved ? 2 * i : i, iv = interleaved ? 2 * i + 1 : i + half;
+      const float a = x[iu], b = x[iv];
       const float2 c = cs[i];
-      x[i] = a * c.x - b * c.y;
-      x[i + half] = b * c.x + a * c.y;
+      x[iu] = a * c.x - b * c.y;
+      x[iv] = b * c.x + a * c.y;
     }
     __syncwarp();
     float sc = 1.0f;
@@ -134,7 +136,7 @@ __global__ void __launch_bounds__(256) rot_norm_prepare_kernel(T* __restrict__ q
 }
 
 extern "C" int qv_rot_norm_prepare(void* q_out, int ld_qo, const float* proj, int ld_p, int q_off, int k_off, int v_off, void* cache,
-                                   const float* cos_sin, int table_rows, int rot, int unit, float eps, const float* head_temp,
+                                   const float* cos_sin, int table_rows, int rot, int interleaved, int unit, float eps, const float* head_temp,
                                    const float* v_first, int ld_vf, float lam, const int* tok_pos, const int* tok_seg,
                                    const int* block_table, int max_blocks, int T, int H, int G, int n, int dv, int page, int dt,
                                    void* stream) {
@@ -150,7 +152,7 @@ extern "C" int qv_rot_norm_prepare(void* q_out, int ld_qo, const float* proj, in
     QV_DISPATCH_DT(dt, TT,
                    rc = qv_launch(rot_norm_prepare_kernel<TT>, dim3(rows), dim3(256), smem, st,
                                   (TT*)((char*)q_out + (size_t)done * ld_qo * esz), ld_qo, proj + (size_t)done * ld_p, ld_p, q_off, k_off,
-                                  v_off, (TT*)cache, (const float2*)cos_sin, table_rows, rot, unit, eps, head_temp,
+                                  v_off, (TT*)cache, (const float2*)cos_sin, table_rows, rot, interleaved, unit, eps, head_temp,
                                   v_first ? v_first + (size_t)done * ld_vf : nullptr, ld_vf, lam, tok_pos + done, tok_seg + done,
                                   block_table, max_blocks, H, G, n, dv, page));
     if (rc) return rc;

@@ -55,6 +55,19 @@ __device__ __forceinline__ float block_sum(float v, float* red /* >= 33 floats *
   return red[32];
 }
 
+// The activations of a gated feed-forward, with the accurate functions: `kind` 0: silu(g) * u, 1: the tanh form of GELU of g, times u,
+// 2: both clamped, g = min(g, limit), u = clamp(u, -limit, limit), then g * sigmoid(slope * g) * (u + 1).
+struct GluAct { int kind; float limit, slope; };
+__device__ __forceinline__ float glu_apply(float g, float u, const GluAct& a) {
+  if (a.kind == 1) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+  if (a.kind == 2) {
+    g = fminf(g, a.limit);
+    u = fminf(fmaxf(u, -a.limit), a.limit);
+    return g / (1.0f + expf(-a.slope * g)) * (u + 1.0f);
+  }
+  return g / (1.0f + expf(-g)) * u;
+}
+
 static inline int qv_launch_status() { return (int)cudaGetLastError(); }
 
 // Programmatic dependent launch: a kernel launched through qv_launch may be scheduled while the

@@ -622,10 +622,10 @@ extern "C" int qv_embed_pos(float* out, const void* table, const void* pos_table
 }
 
 // ---------------------------------------------------------------- gated feed-forward activations
-// out[t, i] = act(gate_i) * up_i; act 0: SiLU, 1: the tanh form of GELU.  gu is [gate | up], or with `interleaved` groups of
+// out[t, i] = glu(gate_i, up_i) (see GluAct in common.cuh).  gu is [gate | up], or with `interleaved` groups of
 // 32 columns: 16 gate values, then the 16 up values of the same features.  Float32 arithmetic.
 template <typename T>
-__global__ void glu_act_kernel(T* __restrict__ out, const T* __restrict__ gu, size_t n, int f, int act, int interleaved) {
+__global__ void glu_act_kernel(T* __restrict__ out, const T* __restrict__ gu, size_t n, int f, GluAct act, int interleaved) {
   pdl_wait();
   pdl_launch_dependents();
   for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < n; idx += (size_t)gridDim.x * blockDim.x) {
@@ -635,17 +635,16 @@ __global__ void glu_act_kernel(T* __restrict__ out, const T* __restrict__ gu, si
     const int ui = interleaved ? gi + 16 : f + i;
     const float g = to_f(gu[t * 2 * f + gi]);
     const float u = to_f(gu[t * 2 * f + ui]);
-    float a;
-    if (act == 1) a = 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
-    else a = g / (1.0f + expf(-g));
-    out[idx] = from_f<T>(a * u);
+    out[idx] = from_f<T>(glu_apply(g, u, act));
   }
 }
 
-extern "C" int qv_glu_act(void* out, const void* gu, int T, int f, int act, int interleaved, int dt, void* stream) {
+// limit, slope: of kind 2
+extern "C" int qv_glu_act(void* out, const void* gu, int T, int f, int kind, float limit, float slope, int interleaved, int dt, void* stream) {
   const size_t n = (size_t)T * f;
   if (n == 0) return 0;
-  if ((act != 0 && act != 1) || (interleaved && (f & 15))) return QV_ERR_UNSUPPORTED;
+  if (kind < 0 || kind > 2 || (interleaved && (f & 15))) return QV_ERR_UNSUPPORTED;
+  const GluAct act = {kind, limit, slope};
   const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
   QV_DISPATCH_DT(dt, TT, return qv_launch(glu_act_kernel<TT>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (TT*)out, (const TT*)gu, n, f, act, interleaved));
   return QV_ERR_UNSUPPORTED;
@@ -722,12 +721,14 @@ extern "C" const char* qv_error_string(int code) {
 
 // ---------------------------------------------------------------- norm on a sublayer's output (post-norm blocks)
 // residual[t] += y[t] * rsqrt(mean(y[t]^2) + eps) * w     (float32; y in the compute type or float32, row stride ld_y)
-// cast[t] = residual[t] in the compute type, if cast is given: what the next sublayer's products read.
+// cast[t] = residual[t] in the compute type, if cast is given: what the next sublayer's products read; with w_next the next
+// sublayer's norm is applied on the way: cast[t] = residual[t] * rsqrt(mean(residual[t]^2) + eps_next) * w_next.
 // One block per row; the sum's order depends on d alone.  VEC: the row of y stays in registers and is read once, four elements
 // at a time (d a multiple of 4, at most 4 * 4 * blockDim elements, rows that start on 16 bytes).
 template <typename TY, typename TO, bool VEC>
 __global__ void __launch_bounds__(256) post_rmsnorm_add_kernel(float* __restrict__ residual, const TY* __restrict__ y, int ld_y,
-                                                              const float* __restrict__ w, float eps, TO* __restrict__ cast, int d) {
+                                                              const float* __restrict__ w, float eps, TO* __restrict__ cast, int d,
+                                                              const float* __restrict__ w_next, float eps_next) {
   __shared__ float red[33];
   pdl_wait();
   pdl_launch_dependents();
@@ -749,6 +750,7 @@ __global__ void __launch_bounds__(256) post_rmsnorm_add_kernel(float* __restrict
     for (int k = 0; k < MAXV; ++k) ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
     const float total = block_sum(ss, red);
     const float sc = 1.0f / sqrtf(total / (float)d + eps);
+    float s2 = 0.f;
 #pragma unroll
     for (int k = 0; k < MAXV; ++k) {
       const int i = threadIdx.x + k * 256;
@@ -757,33 +759,52 @@ __global__ void __launch_bounds__(256) post_rmsnorm_add_kernel(float* __restrict
         const float4 x = make_float4(r[k].x + v[k].x * sc * wv.x, r[k].y + v[k].y * sc * wv.y, r[k].z + v[k].z * sc * wv.z,
                                      r[k].w + v[k].w * sc * wv.w);
         *(float4*)(res + 4 * i) = x;
-        if (cast) store4(cast + (size_t)t * d + 4 * i, x);
+        if (cast && !w_next) store4(cast + (size_t)t * d + 4 * i, x);
+        r[k] = x;
+        s2 += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+      }
+    }
+    if (cast && w_next) {
+      const float sn = 1.0f / sqrtf(block_sum(s2, red) / (float)d + eps_next);
+#pragma unroll
+      for (int k = 0; k < MAXV; ++k) {
+        const int i = threadIdx.x + k * 256;
+        if (i < nvec) {
+          const float4 wv = *(const float4*)(w_next + 4 * i);
+          store4(cast + (size_t)t * d + 4 * i, make_float4(r[k].x * sn * wv.x, r[k].y * sn * wv.y, r[k].z * sn * wv.z, r[k].w * sn * wv.w));
+        }
       }
     }
   } else {
     for (int i = threadIdx.x; i < d; i += blockDim.x) { const float v = to_f(yr[i]); ss = fmaf(v, v, ss); }
     const float total = block_sum(ss, red);
     const float sc = 1.0f / sqrtf(total / (float)d + eps);
+    float s2 = 0.f;
     for (int i = threadIdx.x; i < d; i += blockDim.x) {
       const float x = res[i] + to_f(yr[i]) * sc * w[i];
       res[i] = x;
-      if (cast) cast[(size_t)t * d + i] = from_f<TO>(x);
+      if (cast && !w_next) cast[(size_t)t * d + i] = from_f<TO>(x);
+      s2 = fmaf(x, x, s2);
+    }
+    if (cast && w_next) {                                 // every thread reads back what it wrote itself
+      const float sn = 1.0f / sqrtf(block_sum(s2, red) / (float)d + eps_next);
+      for (int i = threadIdx.x; i < d; i += blockDim.x) cast[(size_t)t * d + i] = from_f<TO>(res[i] * sn * w_next[i]);
     }
   }
 }
 
 extern "C" int qv_post_rmsnorm_add(float* residual, const void* y, int ld_y, const float* w, float eps, void* cast, int T, int d,
-                                   int y_dt, int cast_dt, void* stream) {
+                                   int y_dt, int cast_dt, const float* w_next, float eps_next, void* stream) {
   if (T <= 0 || d <= 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
   const bool vec = d % 4 == 0 && d <= 4 * 4 * 256 && ld_y % 4 == 0 &&
-                   (((uintptr_t)residual | (uintptr_t)y | (uintptr_t)w | (uintptr_t)cast) & 15) == 0;
+                   (((uintptr_t)residual | (uintptr_t)y | (uintptr_t)w | (uintptr_t)cast | (uintptr_t)w_next) & 15) == 0;
 #define LAUNCH_POST(TY, TO)                                                                                                        \
   do {                                                                                                                             \
     if (vec) return qv_launch(post_rmsnorm_add_kernel<TY, TO, true>, dim3(T), dim3(256), 0, st, residual, (const TY*)y, ld_y, w,   \
-                              eps, (TO*)cast, d);                                                                                  \
+                              eps, (TO*)cast, d, w_next, eps_next);                                                                \
     return qv_launch(post_rmsnorm_add_kernel<TY, TO, false>, dim3(T), dim3(256), 0, st, residual, (const TY*)y, ld_y, w, eps,      \
-                     (TO*)cast, d);                                                                                                \
+                     (TO*)cast, d, w_next, eps_next);                                                                              \
   } while (0)
   if (y_dt == QV_DT_F32 && cast_dt == QV_DT_F32) LAUNCH_POST(float, float);
   if (y_dt == QV_DT_BF16 && cast_dt == QV_DT_BF16) LAUNCH_POST(bf16, bf16);

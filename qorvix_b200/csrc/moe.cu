@@ -3,17 +3,21 @@
 //
 // qv_moe_route    logits = Wr h in float32 (fixed summation order), the `top` largest per token (ties: the lower
 //                 index), weights = softmax over the chosen logits only; optionally one more row of the router
-//                 matrix' companion (a scalar gate per token: sigmoid(ws . h)).
+//                 matrix' companion (a scalar gate per token: sigmoid(ws . h)).  With `correction`: scores = softmax over all
+//                 logits, the choice by score + correction, weights = scores * w_scale (not renormalised).
 // qv_moe_route_table  no router: row `token id` of an integer table [vocab, top] lists the token's experts, each weighted 1/top.
 // qv_moe_group    counting sort of the (token, choice) pairs by expert, all on the device (a step never waits
 //                 for the host): row_token[r] = token of sorted row r, slot_row[token * top + j] = its sorted row,
 //                 and a table of row tiles (expert, first row, rows) for the products' grids.
 // qv_moe_experts  CUDA-core products over the grouped rows, float32 multiply-adds with k ascending:
-//                   UP (1):   act[r] = silu(Wg_e h[row_token[r]]) * (Wu_e h[row_token[r]])
+//                   UP (1):   act[r] = glu(Wg_e h[row_token[r]], Wu_e h[row_token[r]])    (GluAct: SiLU, GELU, clamped)
 //                   UP (2):   act[r] = relu(Wu_e h[row_token[r]])^2            (ungated experts)
 //                   DOWN (0): y[r]   = Wd_e act[r]   (float32)
 // qv_moe_combine  delta[t] = (mixer output) * s_mix + (sum_j weight[t, j] * y[slot_row[t, j]] + gate[t] * shared[t]) * s_ff
 //                 in float32, choices summed in the order the router ranked them; s_mix, s_ff: per-feature factors or none.
+//
+// Choices at or beyond the number of experts are identity experts: they take no row in the grouping (slot_row -1) and
+// the sum takes the token's own input for them.
 #include "common.cuh"
 
 #define ROUTE_WARPS 8
@@ -167,7 +171,8 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_logits_tokens_kernel(flo
 template <typename T, typename TW>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(int* __restrict__ top_idx, float* __restrict__ top_w, float* __restrict__ gate_out,
                                                         const T* __restrict__ h, int ld_h, const TW* __restrict__ wr,
-                                                        const TW* __restrict__ wg, int d, int E, int top, const float* __restrict__ pre) {
+                                                        const TW* __restrict__ wg, int d, int E, int top, const float* __restrict__ pre,
+                                                        const float* __restrict__ correction, float w_scale) {
   extern __shared__ float logit[];           // E floats, then the token's d inputs
   pdl_wait();
   pdl_launch_dependents();
@@ -190,6 +195,23 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(int* __rest
   }
   __syncthreads();
   if (warp != 0) return;
+  float* score = xs + d;                     // E floats, with `correction`: the scores, while logit[] holds what the choice is by
+  if (correction) {
+    float mx = -INFINITY, sum = 0.f;
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, logit[e]);
+    mx = warp_max(mx);
+    for (int e = lane; e < E; e += 32) {
+      const float p = expf(logit[e] - mx);
+      score[e] = p;
+      sum += p;
+    }
+    sum = warp_sum(sum);
+    for (int e = lane; e < E; e += 32) {
+      score[e] /= sum;
+      logit[e] = score[e] + correction[e];
+    }
+    __syncwarp();
+  }
   float first = 0.f, denom = 0.f;
   for (int j = 0; j < top; ++j) {
     float best = -INFINITY;
@@ -207,13 +229,18 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(int* __rest
     if (j == 0) first = best;
     const float p = expf(best - first);         // the first choice is the largest: exponents are <= 0
     denom += p;
-    if (lane == 0) {
+    if (lane == 0 && correction) {
+      top_idx[(size_t)t * top + j] = bi < E ? bi : 0;
+      top_w[(size_t)t * top + j] = score[bi < E ? bi : 0] * w_scale;
+      if (bi < E) logit[bi] = -INFINITY;
+    } else if (lane == 0) {
       top_idx[(size_t)t * top + j] = bi < E ? bi : 0;          // (not-a-number logits: still an expert that exists)
       top_w[(size_t)t * top + j] = p;
       if (bi < E) logit[bi] = -INFINITY;
     }
     __syncwarp();
   }
+  if (correction) return;
   for (int j = lane; j < top; j += 32) top_w[(size_t)t * top + j] /= denom;
 }
 
@@ -221,11 +248,12 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(int* __rest
 // 256 tokens over (tokens x groups of eight rows) CTAs, for longer ones over (groups of eight tokens x groups of eight rows); the
 // result is the same whichever kernel forms them (same sums, same order).
 extern "C" int qv_moe_route(int* top_idx, float* top_w, float* gate_out, const void* h, int ld_h, const void* wr, const void* wg,
-                            float* logits_ws, int T, int d, int E, int top, int dt, int w_dt, void* stream) {
+                            float* logits_ws, int T, int d, int E, int top, int dt, int w_dt, const float* correction, float w_scale,
+                            void* stream) {
   if (T <= 0) return 0;
   if (E <= 0 || top <= 0 || top > E || E > 8192) return QV_ERR_UNSUPPORTED;
   cudaStream_t st = (cudaStream_t)stream;
-  const size_t smem = (size_t)(E + d) * sizeof(float);
+  const size_t smem = (size_t)(E + d + (correction ? E : 0)) * sizeof(float);
   if (smem > 48 * 1024) return QV_ERR_TOO_LARGE;
   const bool split = logits_ws && T <= 256;
   // more tokens: the logits by groups of tokens, where the group's rows fit shared memory
@@ -248,7 +276,7 @@ extern "C" int qv_moe_route(int* top_idx, float* top_w, float* gate_out, const v
     }                                                                                                                        \
     return qv_launch(moe_route_kernel<TT, TW>, dim3(T), dim3(ROUTE_WARPS * 32), smem, st, top_idx, top_w, gate_out, (const TT*)h, \
                      ld_h, (const TW*)wr, (const TW*)wg, d, E, top,                                                          \
-                     (split || tokens) ? (const float*)logits_ws : (const float*)nullptr);                                   \
+                     (split || tokens) ? (const float*)logits_ws : (const float*)nullptr, correction, w_scale);              \
   } while (0)
   if (dt == QV_DT_F32 && w_dt == QV_DT_F32) ROUTE(float, float);
   if (dt == QV_DT_BF16 && w_dt == QV_DT_BF16) ROUTE(bf16, bf16);
@@ -293,7 +321,8 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(int* __restrict__ row_t
   int* off = cnt + E;
   for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
-  for (int r = threadIdx.x; r < R; r += blockDim.x) rank_tmp[r] = atomicAdd(&cnt[top_idx[r]], 1);
+  for (int r = threadIdx.x; r < R; r += blockDim.x)
+    if (top_idx[r] < E) rank_tmp[r] = atomicAdd(&cnt[top_idx[r]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int o = 0, n = 0;
@@ -310,6 +339,7 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(int* __restrict__ row_t
   }
   __syncthreads();
   for (int r = threadIdx.x; r < R; r += blockDim.x) {
+    if (top_idx[r] >= E) { slot_row[r] = -1; continue; }       // an identity expert
     const int pos = off[top_idx[r]] + rank_tmp[r];
     slot_row[r] = pos;
     row_token[pos] = r / top;
@@ -345,7 +375,8 @@ extern "C" int qv_moe_group(int* row_token, int* slot_row, int* tiles, const int
 template <typename T, typename TW, int MODE>
 __global__ void __launch_bounds__(256) moe_experts_kernel(void* __restrict__ out_, int ld_out, const T* __restrict__ a, int ld_a,
                                                           const TW* __restrict__ w1, const TW* __restrict__ w2,
-                                                          const int* __restrict__ row_token, const int* __restrict__ tiles, int N, int K) {
+                                                          const int* __restrict__ row_token, const int* __restrict__ tiles, int N, int K,
+                                                          GluAct glu) {
   constexpr bool GATHER = MODE != 0;         // rows of a are gathered, the output is in the compute type
   constexpr bool UP = MODE == 1;             // a second matrix (the gate's partner)
   __shared__ float As[MOE_BK][MOE_BM + 1];
@@ -407,8 +438,7 @@ __global__ void __launch_bounds__(256) moe_experts_kernel(void* __restrict__ out
       const int n = n0 + tx * 4 + c;
       if (n >= N) continue;
       if (UP) {
-        const float g = acc1[r][c];
-        ((T*)out_)[(size_t)(row0 + row) * ld_out + n] = from_f<T>(g / (1.0f + expf(-g)) * acc2[r][c]);
+        ((T*)out_)[(size_t)(row0 + row) * ld_out + n] = from_f<T>(glu_apply(acc1[r][c], acc2[r][c], glu));
       } else if (MODE == 2) {
         const float g = fmaxf(acc1[r][c], 0.f);
         ((T*)out_)[(size_t)(row0 + row) * ld_out + n] = from_f<T>(g * g);
@@ -420,8 +450,11 @@ __global__ void __launch_bounds__(256) moe_experts_kernel(void* __restrict__ out
 }
 
 extern "C" int qv_moe_experts(int up, void* out, int ld_out, const void* a, int ld_a, const void* w1, const void* w2,
-                              const int* row_token, const int* tiles, int R, int E, int N, int K, int dt, int w_dt, void* stream) {
+                              const int* row_token, const int* tiles, int R, int E, int N, int K, int dt, int w_dt, int act, float limit,
+                              float slope, void* stream) {
   if (R <= 0) return 0;
+  if (act < 0 || act > 2) return QV_ERR_UNSUPPORTED;
+  const GluAct glu = {act, limit, slope};
   const int max_tiles = qv_moe_max_tiles(R, E, MOE_BM);
   if (max_tiles > 65535) return QV_ERR_TOO_LARGE;
   dim3 grid((N + MOE_BN - 1) / MOE_BN, max_tiles);
@@ -429,11 +462,11 @@ extern "C" int qv_moe_experts(int up, void* out, int ld_out, const void* a, int 
 #define EXPERTS(TT, TW)                                                                                                        \
   do {                                                                                                                         \
     if (up == 1) return qv_launch(moe_experts_kernel<TT, TW, 1>, grid, dim3(256), 0, st, out, ld_out, (const TT*)a, ld_a, (const TW*)w1, \
-                                  (const TW*)w2, row_token, tiles, N, K);                                                      \
+                                  (const TW*)w2, row_token, tiles, N, K, glu);                                                 \
     if (up == 2) return qv_launch(moe_experts_kernel<TT, TW, 2>, grid, dim3(256), 0, st, out, ld_out, (const TT*)a, ld_a, (const TW*)w1, \
-                                  (const TW*)w2, row_token, tiles, N, K);                                                      \
+                                  (const TW*)w2, row_token, tiles, N, K, glu);                                                 \
     return qv_launch(moe_experts_kernel<TT, TW, 0>, grid, dim3(256), 0, st, out, ld_out, (const TT*)a, ld_a, (const TW*)w1,      \
-                     (const TW*)w2, row_token, tiles, N, K);                                                                   \
+                     (const TW*)w2, row_token, tiles, N, K, glu);                                                              \
   } while (0)
   if (dt == QV_DT_F32 && w_dt == QV_DT_F32) EXPERTS(float, float);
   if (dt == QV_DT_BF16 && w_dt == QV_DT_BF16) EXPERTS(bf16, bf16);
@@ -465,7 +498,8 @@ __device__ __forceinline__ void mma16816(float* c, const uint32_t* a, uint32_t b
 template <int MODE, int BK, int STAGES>
 __global__ void __launch_bounds__(128) moe_experts_tc_kernel(void* __restrict__ out_, int ld_out, const bf16* __restrict__ a, int ld_a,
                                                              const bf16* __restrict__ w1, const bf16* __restrict__ w2,
-                                                             const int* __restrict__ row_token, const int* __restrict__ tiles, int N, int K) {
+                                                             const int* __restrict__ row_token, const int* __restrict__ tiles, int N, int K,
+                                                             GluAct glu) {
   constexpr bool GATHER = MODE != 0;         // modes as in moe_experts_kernel
   constexpr bool UP = MODE == 1;
   constexpr int LD = BK + 8;                 // padded row of a staged tile: ldmatrix without bank conflicts
@@ -556,7 +590,7 @@ __global__ void __launch_bounds__(128) moe_experts_tc_kernel(void* __restrict__ 
           const int n = n0 + wn * 32 + nt * 8 + 2 * (lane & 3) + j;
           if (n >= N) continue;
           const float v = acc1[mt][nt][half * 2 + j];
-          if (UP) ((bf16*)out_)[(size_t)(row0 + r) * ld_out + n] = __float2bfloat16_rn(v / (1.0f + expf(-v)) * acc2[mt][nt][half * 2 + j]);
+          if (UP) ((bf16*)out_)[(size_t)(row0 + r) * ld_out + n] = __float2bfloat16_rn(glu_apply(v, acc2[mt][nt][half * 2 + j], glu));
           else if (MODE == 2) ((bf16*)out_)[(size_t)(row0 + r) * ld_out + n] = __float2bfloat16_rn(fmaxf(v, 0.f) * fmaxf(v, 0.f));
           else ((float*)out_)[(size_t)(row0 + r) * ld_out + n] = v;
         }
@@ -570,8 +604,11 @@ __global__ void __launch_bounds__(128) moe_experts_tc_kernel(void* __restrict__ 
 // several times faster than 64 rows that lie a whole matrix row apart).  The tile table must have been made for tiles
 // of qv_moe_tile_rows(1) rows.  Refuses rows of `a` that do not start on 16 bytes.
 extern "C" int qv_moe_experts_tc(int up, void* out, int ld_out, const void* a, int ld_a, const void* w1, const void* w2,
-                                 const int* row_token, const int* tiles, int R, int E, int N, int K, void* stream) {
+                                 const int* row_token, const int* tiles, int R, int E, int N, int K, int act, float limit, float slope,
+                                 void* stream) {
   if (R <= 0) return 0;
+  if (act < 0 || act > 2) return QV_ERR_UNSUPPORTED;
+  const GluAct glu = {act, limit, slope};
   if ((ld_a & 7) || (((uintptr_t)a | (uintptr_t)w1 | (uintptr_t)w2) & 15)) return QV_ERR_UNSUPPORTED;
   const int max_tiles = qv_moe_max_tiles(R, E, MOE_TC_BM);
   if (max_tiles > 65535) return QV_ERR_TOO_LARGE;
@@ -584,31 +621,37 @@ extern "C" int qv_moe_experts_tc(int up, void* out, int ld_out, const void* a, i
   if (up == 1) {
     cudaFuncSetAttribute(moe_experts_tc_kernel<1, BK, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     return qv_launch(moe_experts_tc_kernel<1, BK, STAGES>, grid, dim3(128), smem, st, out, ld_out, (const bf16*)a, ld_a, (const bf16*)w1,
-                     (const bf16*)w2, row_token, tiles, N, K);
+                     (const bf16*)w2, row_token, tiles, N, K, glu);
   }
   if (up == 2) {
     cudaFuncSetAttribute(moe_experts_tc_kernel<2, BK, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     return qv_launch(moe_experts_tc_kernel<2, BK, STAGES>, grid, dim3(128), smem, st, out, ld_out, (const bf16*)a, ld_a, (const bf16*)w1,
-                     (const bf16*)w2, row_token, tiles, N, K);
+                     (const bf16*)w2, row_token, tiles, N, K, glu);
   }
   cudaFuncSetAttribute(moe_experts_tc_kernel<0, BK, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   return qv_launch(moe_experts_tc_kernel<0, BK, STAGES>, grid, dim3(128), smem, st, out, ld_out, (const bf16*)a, ld_a, (const bf16*)w1,
-                   (const bf16*)w2, row_token, tiles, N, K);
+                   (const bf16*)w2, row_token, tiles, N, K, glu);
 }
 
-// delta [T, d] float32.  mix, shared: [T, d] in the compute type or null; gate [T] float32 or null.
+// delta [T, d] float32.  mix, shared, h (the tokens' inputs, read for identity experts): [T, d] in the compute type or null; gate
+// [T] float32 or null.
 template <typename T>
 __global__ void __launch_bounds__(256) moe_combine_kernel(float* __restrict__ delta, const T* __restrict__ mix, const float* __restrict__ y,
                                                           const int* __restrict__ slot_row, const float* __restrict__ top_w,
                                                           const T* __restrict__ shared, const float* __restrict__ gate, int d, int top,
-                                                          const float* __restrict__ s_mix, const float* __restrict__ s_ff) {
+                                                          const float* __restrict__ s_mix, const float* __restrict__ s_ff,
+                                                          const T* __restrict__ h, int ld_h) {
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x;
   const float g = gate ? gate[t] : 1.f;
   for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < d; i += gridDim.y * blockDim.x) {
     float routed = 0.f;
-    for (int j = 0; j < top; ++j) routed = fmaf(top_w[(size_t)t * top + j], y[(size_t)slot_row[(size_t)t * top + j] * d + i], routed);
+    for (int j = 0; j < top; ++j) {
+      const int r = slot_row[(size_t)t * top + j];
+      const float yv = r >= 0 ? y[(size_t)r * d + i] : (h ? to_f(h[(size_t)t * ld_h + i]) : 0.f);
+      routed = fmaf(top_w[(size_t)t * top + j], yv, routed);
+    }
     float v = routed;
     if (shared) v = fmaf(g, to_f(shared[(size_t)t * d + i]), v);
     if (s_ff) v *= s_ff[i];
@@ -619,10 +662,10 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(float* __restrict__ de
 
 extern "C" int qv_moe_combine(float* delta, const void* mix, const float* y, const int* slot_row, const float* top_w,
                               const void* shared, const float* gate, int T, int d, int top, int dt, const float* s_mix,
-                              const float* s_ff, void* stream) {
+                              const float* s_ff, const void* h, int ld_h, void* stream) {
   if (T <= 0) return 0;
   QV_DISPATCH_DT(dt, TT,
                  return qv_launch(moe_combine_kernel<TT>, dim3(T, T < 256 ? (d + 255) / 256 : 1), dim3(256), 0, (cudaStream_t)stream, delta, (const TT*)mix, y, slot_row,
-                                  top_w, (const TT*)shared, gate, d, top, s_mix, s_ff));
+                                  top_w, (const TT*)shared, gate, d, top, s_mix, s_ff, (const TT*)h, ld_h));
   return QV_ERR_UNSUPPORTED;
 }

@@ -67,13 +67,13 @@ _ARGTYPES = {
     "qv_linear_scan_state_floats": [_I, _I, _I, _I],
     "qv_linear_scan": [_I, _V, _I, _V, _I, _I, _V, _I, _V, _I, _V, _I, _V, _I, _V, _V, _V, _F, _F, _V, _L, _V, _V, _I, _I, _I, _I, _I, _V],
     "qv_gated_group_norm": [_V, _I, _V, _I, _V, _I, _V, _I, _I, _I, _F, _I, _I, _V],
-    "qv_moe_route": [_V, _V, _V, _V, _I, _V, _V, _V, _I, _I, _I, _I, _I, _I, _V],
+    "qv_moe_route": [_V, _V, _V, _V, _I, _V, _V, _V, _I, _I, _I, _I, _I, _I, _V, _F, _V],
     "qv_moe_max_tiles": [_I, _I, _I],
     "qv_moe_tile_rows": [_I],
     "qv_moe_group": [_V, _V, _V, _V, _V, _I, _I, _I, _I, _V],
-    "qv_moe_experts_tc": [_I, _V, _I, _V, _I, _V, _V, _V, _V, _I, _I, _I, _I, _V],
-    "qv_moe_experts": [_I, _V, _I, _V, _I, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _V],
-    "qv_moe_combine": [_V, _V, _V, _V, _V, _V, _V, _I, _I, _I, _I, _V, _V, _V],
+    "qv_moe_experts_tc": [_I, _V, _I, _V, _I, _V, _V, _V, _V, _I, _I, _I, _I, _I, _F, _F, _V],
+    "qv_moe_experts": [_I, _V, _I, _V, _I, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _F, _F, _V],
+    "qv_moe_combine": [_V, _V, _V, _V, _V, _V, _V, _I, _I, _I, _I, _V, _V, _V, _I, _V],
     "qv_moe_route_table": [_V, _V, _V, _V, _I, _I, _I, _I, _V],
     "qv_scale_sum2": [_V, _V, _V, _V, _V, _I, _I, _I, _I, _V],
     "qv_stream_concat": [_V, _V, _V, _V, _I, _I, _I, _I, _V],
@@ -85,15 +85,16 @@ _ARGTYPES = {
     "qv_diff_attention_generic": [_V, _I, _V, _I, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _I, _V],
     "qv_add_tanhnorm": [_V, _V, _V, _V, _V, _F, _V, _I, _I, _I, _I, _I, _V],
     "qv_embed_pos": [_V, _V, _V, _V, _V, _I, _I, _I, _I, _F, _V, _V, _F, _I, _V],
-    "qv_glu_act": [_V, _V, _I, _I, _I, _I, _I, _V],
+    "qv_glu_act": [_V, _V, _I, _I, _I, _F, _F, _I, _I, _V],
+    "qv_gemm_bf16_glu": [_V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _V, _I, _F, _F, _V],
     "qv_sigmoid_gate": [_V, _V, _I, _V, _I, _V, _I, _I, _I, _V],
     "qv_depth_mix": [_V, _V, _V, _L, _V, _I, _V],
     "qv_scale": [_V, _L, _F, _V],
     "qv_channel_gates": [_V, _I, _V, _I, _V, _V, _I, _I, _I, _I, _I, _F, _V, _V],
     "qv_delta_operands": [_V, _V, _V, _V, _I, _V, _I, _V, _I, _V, _I, _I, _I, _I, _I, _F, _F, _V],
-    "qv_post_rmsnorm_add": [_V, _V, _I, _V, _F, _V, _I, _I, _I, _I, _V],
+    "qv_post_rmsnorm_add": [_V, _V, _I, _V, _F, _V, _I, _I, _I, _I, _V, _F, _V],
     "qv_rmsnorm_rows": [_V, _I, _V, _I, _V, _F, _I, _I, _I, _I, _V],
-    "qv_rot_norm_prepare": [_V, _I, _V, _I, _I, _I, _I, _V, _V, _I, _I, _I, _F, _V, _V, _I, _F, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _V],
+    "qv_rot_norm_prepare": [_V, _I, _V, _I, _I, _I, _I, _V, _V, _I, _I, _I, _I, _F, _V, _V, _I, _F, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _V],
     "qv_unit_keys": [_V, _V, _V, _I, _V, _I, _V, _I, _I, _I, _F, _V],
     "qv_channel_scan_state_floats": [_I, _I, _I],
     "qv_channel_scan": [_V, _I, _V, _I, _V, _I, _V, _I, _V, _I, _V, _I, _V, _I, _F, _V, _L, _V, _V, _I, _I, _I, _I, _I, _V],
@@ -101,12 +102,19 @@ _ARGTYPES = {
     "qv_bias_attn_prepare": [_V, _I, _V, _I, _I, _I, _I, _V, _V, _V, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _V],
     "qv_bias_attention_generic": [_V, _I, _V, _I, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _F, _V, _I, _V, _V, _I, _F, _I, _V],
     "qv_bias_attention_mma": [_V, _I, _V, _I, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _F, _V, _I, _V, _I, _F, _V, _I, _I, _V],
+    "qv_talking_attention_generic": [_V, _I, _V, _I, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _F, _F, _V, _V, _I, _V],
+    "qv_talking_attention_mma": [_V, _I, _V, _I, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _V, _V, _V, _V, _I, _I, _I, _V],
+    "qv_head_delta_operands": [_V, _V, _V, _V, _I, _V, _I, _V, _I, _V, _I, _V, _V, _V, _V, _I, _I, _I, _I, _F, _F, _I, _V],
+    "qv_head_delta_coef": [],
+    "qv_head_delta_block": [],
+    "qv_head_delta_state_floats": [_I, _I, _I],
+    "qv_head_delta_scan": [_V, _I, _V, _V, _V, _I, _V, _V, _L, _V, _V, _I, _I, _I, _I, _I, _I, _I, _V],
     "qv_argmax": [_V, _V, _I, _I, _L, _V],
     "qv_sample": [_V, _V, _I, _I, _L, _V, _V, _V, _V, _V, _V, _I, _V, _V, _V, _V],
 }
 _RESTYPES = {"qv_error_string": ctypes.c_char_p, "qv_packed_weight_bytes": c_longlong, "qv_gemm_bf16_split_slot_bytes": c_longlong,
              "qv_linear_scan_state_floats": c_longlong, "qv_latent_tc_workspace_bytes": c_longlong, "qv_diff_partial_floats": c_longlong,
-             "qv_channel_scan_state_floats": c_longlong}
+             "qv_channel_scan_state_floats": c_longlong, "qv_head_delta_state_floats": c_longlong}
 _typed_libs = {}
 
 
@@ -377,16 +385,18 @@ def embed_pos(out, table, pos_table, ids, tok_pos, pos_scale: float = 1.0, weigh
     _check(rc, "embed_pos")
 
 
-GLU_SILU, GLU_GELU_TANH = 0, 1
+GLU_SILU, GLU_GELU_TANH, GLU_CLAMPED = 0, 1, 2
 
 
-def glu_act(out, gu, act: int, interleaved: bool = False) -> None:
-    """out[t, i] = act(gate_i) * up_i; act GLU_SILU or GLU_GELU_TANH; gu is [gate | up], or with `interleaved` groups of
-    32 columns: 16 gate values, then the 16 up values of the same features."""
+def glu_act(out, gu, act: int, interleaved: bool = False, limit: float = 0.0, slope: float = 0.0) -> None:
+    """out[t, i] = act(gate_i) * up_i for GLU_SILU and GLU_GELU_TANH; GLU_CLAMPED: g = min(gate_i, limit), u = up_i clamped to
+    +-limit, out = g * sigmoid(slope * g) * (u + 1).  gu is [gate | up], or with `interleaved` groups of 32 columns: 16 gate
+    values, then the 16 up values of the same features."""
     _need_cuda(out, gu)
     T, f = out.shape
     assert out.dtype == gu.dtype and out.is_contiguous() and gu.is_contiguous() and tuple(gu.shape) == (T, 2 * f)
-    _check(_lib("elementwise").qv_glu_act(_ptr(out), _ptr(gu), T, f, act, 1 if interleaved else 0, dt_code(out.dtype), _stream()), "glu_act")
+    _check(_lib("elementwise").qv_glu_act(_ptr(out), _ptr(gu), T, f, act, float(limit), float(slope), 1 if interleaved else 0, dt_code(out.dtype),
+                                           _stream()), "glu_act")
 
 
 def sigmoid_gate(out, y, g, bias) -> None:
@@ -417,15 +427,18 @@ def scale(x, s: float) -> None:
     _check(_lib("elementwise").qv_scale(_ptr(x), x.numel(), float(s), _stream()), "scale")
 
 
-def post_rmsnorm_add(residual, y, weight, eps: float, cast=None) -> None:
+def post_rmsnorm_add(residual, y, weight, eps: float, cast=None, next_weight=None, next_eps: float = 0.0) -> None:
     """residual (float32 [T, d]) += y / rms(y) * weight, the root mean square over a row of y with eps under the root; y in the
-    compute type or float32 (rows may be strided); `cast`, if given, receives the new residual in its own type."""
-    _need_cuda(residual, y, weight, cast)
+    compute type or float32 (rows may be strided); `cast`, if given, receives the new residual in its own type, with
+    next_weight (float32 [d]) already normed: residual / rms(residual) * next_weight (next_eps under the root)."""
+    _need_cuda(residual, y, weight, cast, next_weight)
+    assert next_weight is None or (cast is not None and next_weight.dtype == torch.float32 and next_weight.numel() == residual.shape[1])
     T, d = residual.shape
     assert residual.dtype == torch.float32 and residual.is_contiguous() and tuple(y.shape) == (T, d) and y.stride(1) == 1
     assert weight.dtype == torch.float32 and weight.numel() == d and (cast is None or (cast.is_contiguous() and cast.shape == residual.shape))
     rc = _lib("elementwise").qv_post_rmsnorm_add(_ptr(residual), _ptr(y), y.stride(0), _ptr(weight), float(eps), _ptr(cast), T, d,
-                                                 dt_code(y.dtype), dt_code(cast.dtype) if cast is not None else F32, _stream())
+                                                 dt_code(y.dtype), dt_code(cast.dtype) if cast is not None else F32, _ptr(next_weight),
+                                                 float(next_eps), _stream())
     _check(rc, "post_rmsnorm_add")
 
 
@@ -782,9 +795,9 @@ def bias_attn_prepare(q_out, proj, q_off, k_off, v_off, bq, bk, bv, cache_layer,
 
 
 def rot_norm_prepare(q_out, proj, q_off, k_off, v_off, cache_layer, cos_sin, rot, unit, eps, head_temp, v_first, lam, ctx, block_table,
-                     H, G, n, dv, page) -> None:
-    """From a float32 product's row [.. q .. k .. v ..]: q and k heads rotated over their first `rot` entries (pairs i, i + rot/2,
-    cos_sin [rows, rot/2, 2] float32), then, with `unit`, divided by their root mean square (eps under the root); q times
+                     H, G, n, dv, page, interleaved: bool = False) -> None:
+    """From a float32 product's row [.. q .. k .. v ..]: q and k heads rotated over their first `rot` entries (pairs i, i + rot/2, or
+    2i, 2i + 1 with `interleaved`; cos_sin [rows, rot/2, 2] float32), then, with `unit`, divided by their root mean square (eps under the root); q times
     head_temp[h] (float32 [H] or None) -> q_out (compute type); v, blended as (1 - lam) v + lam v_first[t] where v_first (float32
     [T, G*dv], a column slice is fine) is given, and k go into the token's cache row [G*n | G*dv]."""
     _need_cuda(q_out, proj, cache_layer, cos_sin, head_temp, v_first, block_table)
@@ -798,7 +811,7 @@ def rot_norm_prepare(q_out, proj, q_off, k_off, v_off, cache_layer, cos_sin, rot
     _i32(block_table, "block_table")
     rc = _lib("bias_attention").qv_rot_norm_prepare(
         _ptr(q_out), q_out.stride(0), _ptr(proj), proj.stride(0), q_off, k_off, v_off, _ptr(cache_layer), _ptr(cos_sin) if rot else None,
-        cos_sin.shape[0] if rot else 1, int(rot), 1 if unit else 0, float(eps), _ptr(head_temp), _ptr(v_first),
+        cos_sin.shape[0] if rot else 1, int(rot), 1 if interleaved else 0, 1 if unit else 0, float(eps), _ptr(head_temp), _ptr(v_first),
         v_first.stride(0) if v_first is not None else 0, float(lam), _ptr(ctx.tok_pos), _ptr(ctx.tok_seg), _ptr(block_table),
         block_table.shape[-1], T, H, G, n, dv, page, dt_code(q_out.dtype), _stream())
     _check(rc, "rot_norm_prepare")
@@ -897,12 +910,151 @@ def bias_attention(out, q, cache_layer, ctx, block_table, H, G, n, dv, page, sca
     bias_attention_generic(out, q, cache_layer, ctx, block_table, H, G, n, dv, page, scale, bucket, bias, gate, factor)
 
 
+# ------------------------------------------------------------------ attention whose heads' weights are mixed
+
+def talking_attention_generic(out, q, cache_layer, ctx, block_table, H, G, n, dv, page, scale, cap, sink, talk) -> None:
+    """out[t, h] = sum_j (sum_g talk[h, g] p_g(t, j)) v_j over the request's pages, p_g the softmax of cap * tanh(q . k * scale / cap)
+    (cap 0: no cap) with exp(sink_g) in its denominator; sink float32 [H], talk float32 [H, H]."""
+    _need_cuda(out, q, cache_layer, block_table, sink, talk)
+    assert q.stride(1) == 1 and out.stride(1) == 1 and q.dtype == out.dtype == cache_layer.dtype
+    assert cache_layer.is_contiguous() and tuple(cache_layer.shape[1:]) == (page, G * (n + dv))
+    assert sink.dtype == talk.dtype == torch.float32 and sink.numel() == H and tuple(talk.shape) == (H, H) and talk.is_contiguous()
+    _i32(block_table, "block_table")
+    rc = _lib("talking_attention").qv_talking_attention_generic(
+        _ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(cache_layer), _ptr(ctx.tok_pos), _ptr(ctx.tok_seg), _ptr(block_table),
+        block_table.shape[-1], q.shape[0], H, G, n, dv, page, float(scale), float(cap), _ptr(sink), _ptr(talk), dt_code(q.dtype), _stream())
+    _check(rc, "talking_attention_generic")
+
+
+def talking_attention_tc(out, q, cache_layer, seg_q_start, seg_pos0, block_table, S, max_q_len, H, G, n, dv, page, scale, cap, sink, talk,
+                         talk_host, slices: int = 1, slice_keys: int = 0, cluster: int = 1) -> bool:
+    """As talking_attention_generic on the tensor cores (bfloat16; up to 16 heads, key and value sizes up to 128 in multiples of 8)
+    for S segments that start at rows seg_q_start[s].  Single tokens (max_q_len 1): keys in `slices` slices of slice_keys that a
+    second launch joins; portions: `cluster` CTAs (1, 2, 4 or 8) share out the keys of 16 tokens.  talk_host: talk as a float32
+    tensor in host memory.  False, nothing written, for sizes it does not take."""
+    if q.dtype != torch.bfloat16 or H > 16 or n % 8 or dv % 8 or n > 128 or dv > 128 or q.stride(0) % 8 or out.stride(0) % 2:
+        return False
+    if q.data_ptr() % 16 or out.data_ptr() % 4:        # 16-byte copies of q, paired stores of the outputs
+        return False
+    _need_cuda(out, q, cache_layer, seg_q_start, seg_pos0, block_table, sink, talk)
+    assert q.stride(1) == 1 and out.stride(1) == 1 and out.dtype == cache_layer.dtype == torch.bfloat16
+    assert cache_layer.is_contiguous() and tuple(cache_layer.shape[1:]) == (page, G * (n + dv))
+    assert sink.dtype == talk.dtype == torch.float32 and sink.numel() == H and tuple(talk.shape) == (H, H) and talk.is_contiguous()
+    assert talk_host.device.type == "cpu" and talk_host.dtype == torch.float32 and talk_host.is_contiguous() and talk_host.numel() == H * H
+    _i32(block_table, "block_table")
+    single = max_q_len == 1
+    partial = torch.empty(S * slices * H * (2 + G * dv), device=q.device, dtype=torch.float32) if single else None
+    rc = _lib("talking_attention").qv_talking_attention_mma(
+        _ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(cache_layer), _ptr(seg_q_start), _ptr(seg_pos0), _ptr(block_table),
+        block_table.shape[-1], S, max_q_len, H, G, n, dv, page, float(scale), float(cap), _ptr(sink), _ptr(talk), _ptr(talk_host),
+        _ptr(partial), slices, slice_keys, cluster, _stream())
+    if rc == -2:
+        return False
+    _check(rc, "talking_attention_mma")
+    if single:
+        add_launches(1)                              # the kernel that joins the slices
+    return True
+
+
+def talking_attention_slices(tokens: int, H: int, values: int, max_ctx: int):
+    """(slices, keys a slice) for single query tokens (a CTA serves a token and a slice; a slice leaves H x `values` partial
+    sums): few tokens still fill the SMs, the slices cover the longest context the step may hold, and their partial sums stay
+    within some hundred megabytes."""
+    keys = 32 if tokens <= 2 else 64 if tokens <= 16 else 128 if tokens <= 64 else 256
+    while tokens * -(-max_ctx // keys) * H * (values + 2) * 4 > 128 << 20 and keys < max_ctx:
+        keys *= 2
+    return max(1, -(-max_ctx // keys)), keys
+
+
+def talking_attention_cluster(tiles: int) -> int:
+    """CTAs that share out the keys of one tile of 16 tokens: few tiles are spread over more SMs."""
+    sms = sm_count()
+    c = 1
+    while c < 8 and tiles * c < 3 * sms // 2:
+        c *= 2
+    return c
+
+
+def talking_attention(out, q, cache_layer, ctx, block_table, H, G, n, dv, page, scale, cap, sink, talk, talk_host) -> None:
+    """Attention with mixed heads for every token of the step (see talking_attention_generic).  bfloat16: the tensor-core kernels
+    where they take the sizes (single tokens, which come first in a step, with their keys in slices; portions in tiles of 16
+    tokens); float32 and other sizes: the CUDA-core kernel."""
+    if q.dtype == torch.bfloat16:
+        S = ctx.num_segments
+        n1 = 0                                        # leading segments of one token (decoded tokens)
+        while n1 < S and ctx.seg_len[n1] == 1:
+            n1 += 1
+        args = (H, G, n, dv, page, scale, cap, sink, talk, talk_host)
+        ok = True
+        if n1:
+            slices, keys = talking_attention_slices(n1, H, G * dv, ctx.max_ctx_len)
+            ok = talking_attention_tc(out, q, cache_layer, ctx.seg_q_start, ctx.seg_pos0, block_table, n1, 1, *args, slices=slices, slice_keys=keys)
+        if ok and n1 < S:
+            lens = ctx.seg_len[n1:]
+            ok = talking_attention_tc(out, q, cache_layer, ctx.seg_q_start[n1:], ctx.seg_pos0[n1:], block_table[n1:], S - n1, max(lens), *args,
+                                      cluster=talking_attention_cluster(sum(-(-m // 16) for m in lens)))
+        if ok:
+            return
+    talking_attention_generic(out, q, cache_layer, ctx, block_table, H, G, n, dv, page, scale, cap, sink, talk)
+
+
+# ------------------------------------------------------------------ delta rule with one decay per head
+
+def head_delta_block(dtype) -> int:
+    """Tokens the recurrence works through together: one for the 32-bit path (every sum's order then depends on the sizes alone)."""
+    return 1 if dtype == torch.float32 else int(_lib("head_delta").qv_head_delta_block())
+
+
+def head_delta_operands(qn, kn, coef, q, k, a, b, rate, dt_bias, ctx, H: int, G: int, n: int, eps: float, q_scale: float, block: int) -> None:
+    """The recurrence's operands (see csrc/head_delta.cu): qn = q / |q| * q_scale, kn = k / |k| per query/key head (dense [T, G*n],
+    |x| = sqrt(sum x^2 + eps)) and coef [T, H, 12] from the decays' and rates' pre-activations a, b (float32 [T, H], column slices
+    are fine), rate = exp(A_log) and dt_bias (float32 [H])."""
+    _need_cuda(qn, kn, coef, q, k, a, b, rate, dt_bias)
+    T = q.shape[0]
+    for x in (qn, kn):
+        assert x.dtype == torch.float32 and x.is_contiguous() and tuple(x.shape) == (T, G * n)
+    for x in (q, k, a, b):
+        assert x.dtype == torch.float32 and x.stride(1) == 1 and x.shape[0] == T
+    assert coef.is_contiguous() and coef.dtype == torch.float32 and tuple(coef.shape) == (T, H, int(_lib("head_delta").qv_head_delta_coef()))
+    assert rate.numel() == dt_bias.numel() == H and rate.dtype == dt_bias.dtype == torch.float32
+    rc = _lib("head_delta").qv_head_delta_operands(_ptr(qn), _ptr(kn), _ptr(coef), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(a),
+                                                   a.stride(0), _ptr(b), b.stride(0), _ptr(rate), _ptr(dt_bias), _ptr(ctx.tok_seg),
+                                                   _ptr(ctx.seg_q_start), T, H, G, n, float(eps), float(q_scale), block, _stream())
+    _check(rc, "head_delta_operands")
+
+
+def head_delta_coef() -> int:
+    """Numbers per token and head in head_delta_operands' coef."""
+    return int(_lib("head_delta").qv_head_delta_coef())
+
+
+def head_delta_state_floats(H: int, dk: int, dv: int) -> int:
+    """How many float32 values head_delta_scan keeps per request for H heads of dk x dv."""
+    return int(_lib("head_delta").qv_head_delta_state_floats(H, dk, dv))
+
+
+def head_delta_scan(out, qn, kn, v, coef, state, ctx, H: int, G: int, dk: int, dv: int, block: int) -> None:
+    """Per request and head: S = g S; S = S + k (beta (v - S^T k))^T; out = S^T q, from head_delta_operands' qn, kn, coef (made for
+    the same `block`); v, out float32 [T, H*dv] (column slices are fine); state [slots, n] float32 is read and left up to date."""
+    _need_cuda(out, qn, kn, v, coef, state)
+    for x in (out, qn, kn, v):
+        assert x.dtype == torch.float32 and x.stride(1) == 1
+    assert state.dtype == torch.float32 and state.stride(-1) == 1 and state.shape[-1] >= head_delta_state_floats(H, dk, dv)
+    rc = _lib("head_delta").qv_head_delta_scan(_ptr(out), out.stride(0), _ptr(qn), _ptr(kn), _ptr(v), v.stride(0), _ptr(coef), _ptr(state),
+                                               state.stride(0), _ptr(ctx.seg_q_start), _ptr(ctx.seg_slot), ctx.num_segments,
+                                               int(ctx.max_q_len), H, G, dk, dv, block, _stream())
+    _check(rc, "head_delta_scan")
+
+
 # ------------------------------------------------------------------ routed feed-forward
 
-def moe_route(top_idx, top_w, gate_out, h, w_router, w_gate) -> None:
+def moe_route(top_idx, top_w, gate_out, h, w_router, w_gate, correction=None, w_scale: float = 1.0) -> None:
     """Per token: router logits in float32, the top choices (top_idx int32 [T, top]) and their weights (softmax
-    over the chosen logits, top_w float32 [T, top]); gate_out [T] = sigmoid(w_gate . h) when w_gate is given."""
-    _need_cuda(top_idx, top_w, gate_out, h, w_router, w_gate)
+    over the chosen logits, top_w float32 [T, top]); gate_out [T] = sigmoid(w_gate . h) when w_gate is given.  With
+    `correction` (float32, a number per row of the router): scores are the softmax over all logits, the choice goes by
+    score + correction and the weights are the chosen scores times w_scale."""
+    _need_cuda(top_idx, top_w, gate_out, h, w_router, w_gate, correction)
+    assert correction is None or (correction.dtype == torch.float32 and correction.is_contiguous() and correction.numel() == w_router.shape[0])
     T, d = h.shape
     E, top = w_router.shape[0], top_idx.shape[1]
     assert h.stride(1) == 1 and w_router.is_contiguous() and w_router.shape[1] == d and top_idx.is_contiguous() and top_w.is_contiguous()
@@ -910,7 +1062,8 @@ def moe_route(top_idx, top_w, gate_out, h, w_router, w_gate) -> None:
     few = T <= 256 or (d % 4 == 0 and 8 * d * 4 <= 160 * 1024)
     ws = torch.empty(T * (E + 1), device=h.device, dtype=torch.float32) if few else None
     rc = _lib("moe").qv_moe_route(_ptr(top_idx), _ptr(top_w), _ptr(gate_out), _ptr(h), h.stride(0), _ptr(w_router), _ptr(w_gate),
-                                  _ptr(ws), T, d, E, top, dt_code(h.dtype), dt_code(w_router.dtype), _stream())
+                                  _ptr(ws), T, d, E, top, dt_code(h.dtype), dt_code(w_router.dtype), _ptr(correction), float(w_scale),
+                                  _stream())
     _check(rc, "moe_route")
     if few:
         add_launches(1)
@@ -926,7 +1079,8 @@ def moe_max_tiles(rows: int, experts: int, tile_rows: int) -> int:
 
 
 def moe_group(row_token, slot_row, tiles, top_idx, scratch, experts: int, tile_rows: int) -> None:
-    """Sorts the (token, choice) pairs by expert on the device and lists the tiles of `tile_rows` rows; see csrc/moe.cu."""
+    """Sorts the (token, choice) pairs by expert on the device and lists the tiles of `tile_rows` rows; choices at or beyond
+    `experts` (identity experts) take no row: their slot_row is -1; see csrc/moe.cu."""
     _need_cuda(row_token, slot_row, tiles, top_idx, scratch)
     T, top = top_idx.shape
     rc = _lib("moe").qv_moe_group(_ptr(row_token), _ptr(slot_row), _ptr(tiles), _ptr(top_idx), _ptr(scratch), T, top, experts,
@@ -944,7 +1098,7 @@ def moe_pack_experts(w: torch.Tensor) -> torch.Tensor:
     return w.view(E, Np // 64, 64, Kp // 64, 64).permute(0, 1, 3, 2, 4).contiguous()
 
 
-def moe_experts_tc(up, out, a, p1, p2, row_token, tiles) -> None:
+def moe_experts_tc(up, out, a, p1, p2, row_token, tiles, act: int = GLU_SILU, limit: float = 0.0, slope: float = 0.0) -> None:
     """The experts' products on the tensor cores (bfloat16); up as for moe_experts.  p1, p2: matrices packed by moe_pack_experts; the sizes
     follow from out [R, N] and a [., K]; the tile table was made for tiles of moe_tile_rows(True) rows."""
     _need_cuda(out, a, p1, p2, row_token, tiles)
@@ -955,13 +1109,13 @@ def moe_experts_tc(up, out, a, p1, p2, row_token, tiles) -> None:
     assert p1.is_contiguous() and tuple(p1.shape[1:]) == (-(-N // 64), -(-K // 64), 64, 64) and R == row_token.numel()
     assert out.dtype == (torch.bfloat16 if up else torch.float32)
     rc = _lib("moe").qv_moe_experts_tc(int(up), _ptr(out), out.stride(0), _ptr(a), a.stride(0), _ptr(p1), _ptr(p2),
-                                       _ptr(row_token), _ptr(tiles), R, E, N, K, _stream())
+                                       _ptr(row_token), _ptr(tiles), R, E, N, K, act, float(limit), float(slope), _stream())
     _check(rc, "moe_experts_tc")
 
 
-def moe_experts(up, out, a, w1, w2, row_token, tiles) -> None:
+def moe_experts(up, out, a, w1, w2, row_token, tiles, act: int = GLU_SILU, limit: float = 0.0, slope: float = 0.0) -> None:
     """The experts' products over the grouped rows on the CUDA cores (float32 multiply-adds, k ascending).
-    up True or 1: out[r] = silu(w1[e] x) * (w2[e] x) with x = a[row_token[r]]; 2: out[r] = relu(w1[e] x)^2 (ungated
+    up True or 1: out[r] = silu(w1[e] x) * (w2[e] x) with x = a[row_token[r]] (act, limit, slope: another gated activation, see glu_act); 2: out[r] = relu(w1[e] x)^2 (ungated
     experts, w2 None); False or 0: out[r] (float32) = w1[e] a[r].
     w1, w2: [E, N, K]; the tile table was made for tiles of moe_tile_rows(False) rows."""
     _need_cuda(out, a, w1, w2, row_token, tiles)
@@ -970,7 +1124,8 @@ def moe_experts(up, out, a, w1, w2, row_token, tiles) -> None:
     assert w1.is_contiguous() and a.stride(1) == 1 and out.stride(1) == 1 and a.shape[1] == K and out.shape == (R, N)
     assert out.dtype == (a.dtype if up else torch.float32)
     rc = _lib("moe").qv_moe_experts(int(up), _ptr(out), out.stride(0), _ptr(a), a.stride(0), _ptr(w1), _ptr(w2),
-                                    _ptr(row_token), _ptr(tiles), R, E, N, K, dt_code(a.dtype), dt_code(w1.dtype), _stream())
+                                    _ptr(row_token), _ptr(tiles), R, E, N, K, dt_code(a.dtype), dt_code(w1.dtype), act, float(limit),
+                                    float(slope), _stream())
     _check(rc, "moe_experts")
 
 
@@ -984,20 +1139,22 @@ def moe_route_table(top_idx, top_w, table, ids, experts: int) -> None:
     _check(rc, "moe_route_table")
 
 
-def moe_combine(delta, mix, y, slot_row, top_w, shared, gate, mix_scale=None, ff_scale=None) -> None:
+def moe_combine(delta, mix, y, slot_row, top_w, shared, gate, mix_scale=None, ff_scale=None, identity_in=None) -> None:
     """delta (float32) = mix * mix_scale + (sum_j top_w[t, j] * y[slot_row[t, j]] + gate[t] * shared[t]) * ff_scale; mix,
-    shared, gate and the per-feature scales (float32 [d]) may be None."""
-    _need_cuda(delta, mix, y, slot_row, top_w, shared, gate, mix_scale, ff_scale)
+    shared, gate and the per-feature scales (float32 [d]) may be None.  identity_in: the tokens' inputs [T, d], taken for y where
+    slot_row is -1 (identity experts)."""
+    _need_cuda(delta, mix, y, slot_row, top_w, shared, gate, mix_scale, ff_scale, identity_in)
     for sc in (mix_scale, ff_scale):
         assert sc is None or (sc.dtype == torch.float32 and sc.is_contiguous() and sc.numel() == delta.shape[1])
     T, d = delta.shape
     assert delta.dtype == torch.float32 and delta.is_contiguous() and y.dtype == torch.float32 and y.is_contiguous()
-    ref = mix if mix is not None else shared
+    ref = mix if mix is not None else shared if shared is not None else identity_in
+    assert identity_in is None or (identity_in.dtype == ref.dtype and identity_in.stride(1) == 1 and identity_in.shape == delta.shape)
     for t in (mix, shared):
         assert t is None or (t.is_contiguous() and t.shape == delta.shape and t.dtype == ref.dtype)
     rc = _lib("moe").qv_moe_combine(_ptr(delta), _ptr(mix), _ptr(y), _ptr(slot_row), _ptr(top_w), _ptr(shared), _ptr(gate), T, d,
                                     top_w.shape[1], dt_code(ref.dtype) if ref is not None else F32, _ptr(mix_scale), _ptr(ff_scale),
-                                    _stream())
+                                    _ptr(identity_in), identity_in.stride(0) if identity_in is not None else 0, _stream())
     _check(rc, "moe_combine")
 
 
@@ -1262,12 +1419,33 @@ def glu_epilogue(act: int) -> int:
     return 2 if act == GLU_GELU_TANH else 1
 
 
-def gemm_swiglu(out, x, w_interleaved, packed=None, n: int = 0, act: int = 0) -> None:
-    """out[M,f] = act(x Wg^T) * (x Wu^T) (act GLU_SILU or GLU_GELU_TANH) with gate and up rows interleaved in groups
-    of 16 in w_interleaved [2f, K]: one tensor-core kernel when it takes the shape, else the product followed
-    by the activation kernel."""
+def gemm_bf16_glu(out, x, w_interleaved, packed, n: int, act: int, limit: float, slope: float) -> bool:
+    """The gate/up product on the tensor cores with an activation that has constants (see glu_act) in its epilogue; False,
+    nothing written, for a product the kernel does not take."""
+    _need_cuda(out, x, w_interleaved, packed)
+    M, K = x.shape
+    if x.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or (packed is None and (w_interleaved is None or w_interleaved.dtype != torch.bfloat16)):
+        return False
+    assert tuple(out.shape) == (M, n // 2) and x.stride(1) == 1 and out.stride(1) == 1
+    st = _gemm_buffers(x.device)
+    rc = _lib("gemm_bf16").qv_gemm_bf16_glu(_ptr(out), _ptr(x), _ptr(w_interleaved), _ptr(packed), M, n, K, x.stride(0),
+                                            w_interleaved.stride(0) if w_interleaved is not None else K, out.stride(0), _ptr(st["err"]), act,
+                                            float(limit), float(slope), _stream())
+    if rc == -2:
+        return False
+    _check(rc, "gemm_bf16_glu")
+    return True
+
+
+def gemm_swiglu(out, x, w_interleaved, packed=None, n: int = 0, act: int = 0, limit: float = 0.0, slope: float = 0.0) -> None:
+    """out[M,f] = act(x Wg^T) * (x Wu^T) (act GLU_SILU or GLU_GELU_TANH; GLU_CLAMPED with limit and slope: see glu_act) with gate
+    and up rows interleaved in groups of 16 in w_interleaved [2f, K]: one tensor-core kernel when it takes the shape, else
+    the product followed by the activation kernel."""
     n = n or w_interleaved.shape[0]
-    if x.dtype == torch.bfloat16 and out.dtype == torch.bfloat16:
+    if act == GLU_CLAMPED:
+        if gemm_bf16_glu(out, x, w_interleaved, packed, n, act, limit, slope):
+            return
+    elif x.dtype == torch.bfloat16 and out.dtype == torch.bfloat16:
         if packed is not None and gemm_bf16_packed(out, x, packed, n, swiglu=glu_epilogue(act)):
             return
         if (w_interleaved is not None and w_interleaved.dtype == torch.bfloat16
@@ -1275,7 +1453,7 @@ def gemm_swiglu(out, x, w_interleaved, packed=None, n: int = 0, act: int = 0) ->
             return
     gu = torch.empty((x.shape[0], n), device=x.device, dtype=out.dtype)
     gemm(gu, x, w_interleaved, packed, n)
-    glu_act(out, gu, act, interleaved=True)
+    glu_act(out, gu, act, interleaved=True, limit=limit, slope=slope)
 
 
 def attention_prefill_bf16(out, q, cache_layer, seg_q_start, seg_pos0, block_table, S, max_q_len, H, Hkv, hd, page,

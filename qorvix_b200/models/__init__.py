@@ -3,4 +3,5 @@ from . import deganex        # registers "Deganex"
 from . import lotirax        # registers "Lotirax"
 from . import tubazen        # registers "Tubazen"
 from . import lugizen        # registers "Lugizen"
+from . import nedasun        # registers "Nedasun"
 from .text_model import TextModel

@@ -101,8 +101,10 @@ class TextModel:
             if self.loop is not None and run in self.loop.pass_of:
                 residual, pending = self.loop.forward(run, residual, pending, x0), None
             # which norm reads the stream after this block (a block that can prepares that norm's input);
-            # none after the last block: the final norm gathers the wanted rows
+            # none after the last block: the final norm gathers the wanted rows; none either where the stream changes between the runs
             nxt = self.blocks[self.order[run + 1]] if run + 1 < len(self.order) else None
+            if self.depth is not None or (self.loop is not None and run + 1 in self.loop.pass_of):
+                nxt = None
             ctx.next_norm = nxt.first_norm() if hasattr(nxt, "first_norm") else None
             residual, pending = self.blocks[li].forward(residual, pending, ctx, self._view(cache, run))
             if self.depth is not None:
@@ -130,3 +132,4 @@ class _BlockView:
         self.mixer_scale, self.ffn_scale = getattr(layer, "mixer_scale", None), getattr(layer, "ffn_scale", None)
         self.residual_mult = getattr(layer, "residual_mult", 1.0)
         self.mixer_gate, self.ffn_gate = getattr(layer, "mixer_gate", None), getattr(layer, "ffn_gate", None)
+        self.mixer_post_norm, self.ffn_post_norm = getattr(layer, "mixer_post_norm", None), getattr(layer, "ffn_post_norm", None)

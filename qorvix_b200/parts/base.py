@@ -62,6 +62,20 @@ class PreNormed:
         return self.norm.add_norm(self.residual, None)
 
 
+@dataclass
+class ReadyNormed(PreNormed):
+    """The input of a norm's part with the norm already applied (`rows`, the compute type), left by a block whose last pass over the
+    stream could apply it; the stream is whole.  Parts take the rows as they are: nothing is left to finish in a product."""
+    scaled: torch.Tensor = None
+    stats: object = None
+    norm: object = None
+    residual: torch.Tensor = None
+    rows: torch.Tensor = None
+
+    def materialise(self) -> torch.Tensor:
+        return self.rows
+
+
 class Mixer:
     def cache_spec(self):
         return None

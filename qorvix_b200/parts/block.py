@@ -1,13 +1,14 @@
 """Block arrangements.  'pre_norm' is the reference's (runtime/src/text_model.cpp:146-168):
     x += mixer(norm(x));  x += feed_forward(norm(x))
 The residual stream is float32.  A block hands the feed-forward's output on as a pending
-delta, which the next norm adds in its own pass.  'post_norm' puts the norms on the parts' outputs instead."""
+delta, which the next norm adds in its own pass.  'post_norm' puts the norms on the parts' outputs instead, 'sandwich_norm'
+on both sides of a part."""
 from __future__ import annotations
 
 import torch
 
 from ..csrc import ops
-from .base import Block, PreNormed
+from .base import Block, PreNormed, ReadyNormed
 from .linear import Linear
 from .registry import build_part, register_part
 
@@ -45,6 +46,8 @@ class PreNormBlock(Block):
     def _normed(norm, part, residual, pending):
         """The input of `part`: the PreNormed as it is when it was made for this norm and the part takes
         one, else the normed rows."""
+        if isinstance(pending, ReadyNormed) and pending.norm is norm:
+            return pending.rows
         if isinstance(pending, PreNormed) and pending.norm is norm and getattr(part, "folds_norms", False):
             return pending
         return norm.add_norm(residual, pending)
@@ -220,7 +223,58 @@ class PostNormBlock(Block):
         return None                              # no norm reads the stream
 
 
+class SandwichNormBlock(Block):
+    """x += post_a(mixer(norm_a(x)));  x += post_b(feed_forward(norm_b(x))).  The pass that adds a part's normed output to the float32
+    stream also applies the norm of the part after it (of this block, or the one the next block starts with), so the stream is
+    read and written once a part; the next block finds its first part's input as a ReadyNormed."""
+
+    def __init__(self, spec, source, rt):
+        self.rt = rt
+        self.mixer = build_part("mixer", spec.mixer, source, rt)
+        self.feed_forward = build_part("feed_forward", spec.feed_forward, source, rt)
+        self.mixer_norm, self.mixer_post = self._norms(self.mixer, spec.mixer_norm, spec.mixer_post_norm, source, rt)
+        self.ffn_norm, self.ffn_post = self._norms(self.feed_forward, spec.ffn_norm, spec.ffn_post_norm, source, rt)
+
+    @staticmethod
+    def _norms(part, before, after, source, rt):
+        if part is None:
+            return None, None
+        pre, post = build_part("norm", before, source, rt), build_part("norm", after, source, rt)
+        if not hasattr(post, "add_normed"):
+            raise ValueError("a sandwich-norm block needs norms that can be added to the stream (add_normed)")
+        return pre, post
+
+    def _input(self, norm, residual, pending):
+        if isinstance(pending, ReadyNormed) and pending.norm is norm:
+            return pending.rows
+        return norm.add_norm(residual, pending)
+
+    def _add(self, post, residual, y, nxt):
+        """The stream takes the normed output; `nxt` (the norm that reads the stream next, or None) is applied in the same pass
+        where it is an RMS norm over the stream."""
+        if not _folds(nxt) or nxt.size != residual.shape[1]:
+            post.add_normed(residual, y)
+            return None
+        rows = torch.empty(residual.shape, device=residual.device, dtype=self.rt.dtype)
+        post.add_normed(residual, y, cast=rows, next_norm=nxt)
+        return ReadyNormed(norm=nxt, residual=residual, rows=rows)
+
+    def forward(self, residual, pending, ctx, cache):
+        after = getattr(ctx, "next_norm", None)
+        if self.mixer is not None:
+            y = self.mixer.forward(self._input(self.mixer_norm, residual, pending), ctx, cache)
+            pending = self._add(self.mixer_post, residual, y, self.ffn_norm if self.feed_forward is not None else after)
+        if self.feed_forward is not None:
+            y = self.feed_forward.forward(self._input(self.ffn_norm, residual, pending), ctx)
+            pending = self._add(self.ffn_post, residual, y, after)
+        return residual, pending
+
+    def first_norm(self):
+        return self.mixer_norm if self.mixer is not None else self.ffn_norm
+
+
 register_part("block", "pre_norm", PreNormBlock)
+register_part("block", "sandwich_norm", SandwichNormBlock)
 register_part("block", "post_norm", PostNormBlock)
 register_part("block", "gated_pre_norm", GatedPreNormBlock)
 register_part("block", "parallel", ParallelBlock)

@@ -1,5 +1,6 @@
 """Mixers whose state per request is a matrix per head that decays channel by channel: gated linear attention, the
-generalized delta rule and the delta rule that removes from the decayed state.  Both are the recurrence S = diag(w) S - (a u)(u^T S) + k v^T, y = S^T q (csrc/channel_scan.cu; the
+generalized delta rule and the delta rule that removes from the decayed state, and the last one with a single decay per
+head, which has kernels of its own (csrc/head_delta.cu).  The others are the recurrence S = diag(w) S - (a u)(u^T S) + k v^T, y = S^T q (csrc/channel_scan.cu; the
 removal term only for the delta rule).  The state is float32, lives in the cache manager's request slots (zeroed at
 admission) and is carried from step to step, so a prompt may be cut anywhere.  Decays, removal rates, unit keys, the
 recurrence and the norms behind it are float32 on every path; the projections leave float32 sums."""
@@ -173,6 +174,64 @@ class ChannelDelta(SharedIOMixer):
         ops.head_norm_gate(out, y, gate, self.norm, H, self.spec.eps, ops.HEAD_GATE_SIGMOID, factor)
 
 
+class HeadDelta(SharedIOMixer):
+    """Delta rule with one decay per head whose removal reads the decayed state; q, k and v pass a short convolution with SiLU, the
+    heads' outputs are normed, weighted and gated with SiLU of a projection.  Every projection of the input is a row block of
+    one product with float32 sums."""
+
+    def __init__(self, spec, source, rt):
+        self.spec, self.rt = spec, rt
+        self.H, self.G, self.dk, self.dv = spec.num_heads, spec.num_kv_heads, spec.key_dim, spec.value_dim
+        if self.H % self.G:
+            raise ValueError(f"num_heads {self.H} is not a multiple of num_kv_heads {self.G}")
+        H, G, dk, dv = self.H, self.G, self.dk, self.dv
+        names = (spec.q_proj, spec.k_proj, spec.v_proj, spec.gate_proj, spec.beta_proj, spec.a_proj)
+        self._w_in = stack_rows([source.get(n) for n in names])
+        self._w_out = source.get(spec.o_proj)
+        self.conv_ch = 2 * G * dk + H * dv
+        self.in_rows = self.conv_ch + H * dv + 2 * H
+        self.out_cols = H * dv
+        self.taps = int(spec.conv_taps)
+        self.conv_w = torch.cat([source.get(n + ".conv", dtype=torch.float32) for n in (spec.q_proj, spec.k_proj, spec.v_proj)], dim=0).contiguous()
+        if tuple(self.conv_w.shape) != (self.conv_ch, self.taps):
+            raise ValueError(f"the convolutions' weights have shape {tuple(self.conv_w.shape)}, not {(self.conv_ch, self.taps)}")
+        self.dt_bias = source.get(spec.dt_bias, dtype=torch.float32).reshape(-1).contiguous()
+        self.rate = torch.exp(source.get(spec.a_log, dtype=torch.float32).double()).float().reshape(-1).contiguous()
+        self.norm = source.get(spec.norm, dtype=torch.float32).repeat(H).contiguous()           # one weight for all heads
+        self.block = ops.head_delta_block(rt.dtype)
+
+    def cache_spec(self):
+        return (FixedStateSpec((ops.head_delta_state_floats(self.H, self.dk, self.dv),), "float32"),
+                FixedStateSpec((max(1, (self.taps - 1) * self.conv_ch),), "float32"))
+
+    def in_weights(self):
+        return self._w_in
+
+    def out_weight(self):
+        return self._w_out
+
+    def release_weights(self):
+        self._w_in = self._w_out = None
+
+    def heads_out(self, proj, ctx, cache, out, factor=1.0):
+        H, G, dk, dv, C = self.H, self.G, self.dk, self.dv, self.conv_ch
+        T, dev = proj.shape[0], proj.device
+        g0, b0 = C, C + H * dv
+        a0 = b0 + H
+        scan_state, conv_state = cache.views[0].tensor, cache.views[1].tensor
+        conv = torch.empty((T, C), device=dev, dtype=torch.float32)
+        ops.conv_state(conv, proj[:, :C], self.conv_w, None, conv_state, ctx, act=True)
+        qn = torch.empty((T, G * dk), device=dev, dtype=torch.float32)
+        kn = torch.empty_like(qn)
+        coef = torch.empty((T, H, ops.head_delta_coef()), device=dev, dtype=torch.float32)
+        ops.head_delta_operands(qn, kn, coef, conv[:, : G * dk], conv[:, G * dk: 2 * G * dk], proj[:, a0: a0 + H], proj[:, b0: b0 + H],
+                                self.rate, self.dt_bias, ctx, H, G, dk, self.spec.key_eps, dk ** -0.5, self.block)
+        y = torch.empty((T, H * dv), device=dev, dtype=torch.float32)
+        ops.head_delta_scan(y, qn, kn, conv[:, 2 * G * dk:], coef, scan_state, ctx, H, G, dk, dv, self.block)
+        ops.head_norm_gate(out, y, proj[:, g0:b0], self.norm, H, self.spec.eps, ops.HEAD_GATE_SILU, factor)
+
+
+register_part("mixer", "head_delta", HeadDelta)
 register_part("mixer", "channel_delta", ChannelDelta)
 register_part("mixer", "gla", GLA)
 register_part("mixer", "delta_rule", DeltaRule)

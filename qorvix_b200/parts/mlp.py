@@ -1,6 +1,6 @@
 """Gated feed-forward: down(act(gate x) * up x), dense, no bias; act is SiLU
-(reference: runtime/src/text_model.cpp:162-168, runtime/src/ops.cpp:96-100) or the tanh form of GELU.  gate and up
-are one fused projection."""
+(reference: runtime/src/text_model.cpp:162-168, runtime/src/ops.cpp:96-100) or the tanh form of GELU, or both halves are
+clamped first (SwiGLUSpec).  gate and up are one fused projection."""
 from __future__ import annotations
 
 import torch
@@ -9,6 +9,9 @@ from ..csrc import ops
 from .base import FeedForward, PreNormed
 from .linear import Linear
 from .registry import register_part
+
+
+GLU_ACTIVATIONS = {"silu": ops.GLU_SILU, "gelu_tanh": ops.GLU_GELU_TANH, "clamped": ops.GLU_CLAMPED}
 
 
 class SwiGLU(FeedForward):
@@ -20,11 +23,12 @@ class SwiGLU(FeedForward):
         # When the width allows, gate and up rows are interleaved in groups of 16 (16 gate rows, the 16
         # up rows of the same features, ...), so that one tile of the product holds both halves of a
         # feature and the activation is applied in the product's epilogue.
-        acts = {"silu": ops.GLU_SILU, "gelu_tanh": ops.GLU_GELU_TANH}
+        acts = GLU_ACTIVATIONS
         name = getattr(spec, "activation", "silu")
         if name not in acts:
             raise ValueError(f"unknown activation '{name}' (known: {', '.join(acts)})")
         self.act = acts[name]
+        self.limit, self.slope = float(getattr(spec, "limit", 0.0)), float(getattr(spec, "slope", 0.0))
         self.interleaved = self.f % 16 == 0
         if self.interleaved:
             k = g.shape[1]
@@ -45,15 +49,16 @@ class SwiGLU(FeedForward):
         act = None
         if isinstance(x, PreNormed):
             act = torch.empty((x.scaled.shape[0], self.f), device=x.scaled.device, dtype=self.rt.dtype)
-            if not (self.interleaved and self.gate_up.forward_prenormed(x, act, swiglu=ops.glu_epilogue(self.act))):
+            if not (self.interleaved and self.act != ops.GLU_CLAMPED and self.gate_up.forward_prenormed(x, act, swiglu=ops.glu_epilogue(self.act))):
                 act, x = None, x.materialise()
         if act is None:
             act = torch.empty((x.shape[0], self.f), device=x.device, dtype=self.rt.dtype)
             if self.interleaved:
-                ops.gemm_swiglu(act, x, self.gate_up.weight, self.gate_up.packed, self.gate_up.out_features, act=self.act)
+                ops.gemm_swiglu(act, x, self.gate_up.weight, self.gate_up.packed, self.gate_up.out_features, act=self.act,
+                               limit=self.limit, slope=self.slope)
             else:
                 gu = self.gate_up(x, out_dtype=self.rt.dtype)
-                ops.glu_act(act, gu, self.act)
+                ops.glu_act(act, gu, self.act, limit=self.limit, slope=self.slope)
         if residual is not None and next_norm is not None:
             pre = self.down.forward_to_stream(act, residual, next_norm)
             if pre is not None:

@@ -1,4 +1,4 @@
-"""Routed feed-forward (mixture of experts) with an optional shared expert.  The router runs in float32;
+"""Routed feed-forward (mixture of experts) with an optional shared expert and identity experts.  The router runs in float32;
 tokens are grouped by expert on the device, the experts' products run over the grouped rows, and one
 kernel forms the weighted sum in token order, adds the shared expert (scaled by its per-token gate) and,
 if given, the output of the part that ran beside it (csrc/moe.cu)."""
@@ -8,6 +8,7 @@ import torch
 
 from ..csrc import ops
 from .base import FeedForward
+from .mlp import GLU_ACTIVATIONS
 from .registry import build_part, register_part
 
 
@@ -28,7 +29,12 @@ class RoutedFeedForward(FeedForward):
         if self.tensor_cores:
             self.w_gate, self.w_up, self.w_down = (ops.moe_pack_experts(w) for w in (self.w_gate, self.w_up, self.w_down))
         self.shared = build_part("feed_forward", spec.shared, source, rt)
-        self.shared_gate = source.get(spec.shared_gate).to(self.router.dtype).reshape(-1) if spec.shared is not None else None
+        gated = spec.shared is not None and spec.shared_gate is not None
+        self.shared_gate = source.get(spec.shared_gate).to(self.router.dtype).reshape(-1) if gated else None
+        self.correction = source.get(spec.correction, dtype=torch.float32).reshape(-1).contiguous() if spec.correction is not None else None
+        if spec.activation not in GLU_ACTIVATIONS:
+            raise ValueError(f"unknown activation '{spec.activation}' (known: {', '.join(GLU_ACTIVATIONS)})")
+        self.glu = dict(act=GLU_ACTIVATIONS[spec.activation], limit=float(spec.limit), slope=float(spec.slope))
 
     def forward(self, x, ctx, add=None, add_scale=None, scale=None):
         s = self.spec
@@ -37,8 +43,8 @@ class RoutedFeedForward(FeedForward):
         R = T * s.top
         top_idx = torch.empty((T, s.top), device=dev, dtype=torch.int32)
         top_w = torch.empty((T, s.top), device=dev, dtype=torch.float32)
-        gate = torch.empty(T, device=dev, dtype=torch.float32) if self.shared is not None else None
-        ops.moe_route(top_idx, top_w, gate, x, self.router, self.shared_gate)
+        gate = torch.empty(T, device=dev, dtype=torch.float32) if self.shared_gate is not None else None
+        ops.moe_route(top_idx, top_w, gate, x, self.router, self.shared_gate, correction=self.correction, w_scale=s.route_scale)
         tc = self.tensor_cores
         tile_rows = ops.moe_tile_rows(tc)
         ints = torch.empty(3 * R + 3 * ops.moe_max_tiles(R, s.experts, tile_rows), device=dev, dtype=torch.int32)
@@ -47,14 +53,15 @@ class RoutedFeedForward(FeedForward):
         act = torch.empty((R, s.expert_ff), device=dev, dtype=x.dtype)
         y = torch.empty((R, d), device=dev, dtype=torch.float32)
         if tc:
-            ops.moe_experts_tc(True, act, x, self.w_gate, self.w_up, row_token, tiles)
+            ops.moe_experts_tc(True, act, x, self.w_gate, self.w_up, row_token, tiles, **self.glu)
             ops.moe_experts_tc(False, y, act, self.w_down, None, row_token, tiles)
         else:
-            ops.moe_experts(True, act, x, self.w_gate, self.w_up, row_token, tiles)
+            ops.moe_experts(True, act, x, self.w_gate, self.w_up, row_token, tiles, **self.glu)
             ops.moe_experts(False, y, act, self.w_down, None, row_token, tiles)
         shared = self.shared.forward(x, ctx) if self.shared is not None else None
         delta = torch.empty((T, d), device=dev, dtype=torch.float32)
-        ops.moe_combine(delta, add, y, slot_row, top_w, shared, gate, mix_scale=add_scale, ff_scale=scale)
+        ops.moe_combine(delta, add, y, slot_row, top_w, shared, gate, mix_scale=add_scale, ff_scale=scale,
+                        identity_in=x if s.identity else None)
         return delta
 
 

@@ -38,10 +38,13 @@ class RMSNorm(Norm):
         return out
 
 
-    def add_normed(self, residual, y, cast=None):
-        """residual (float32) += rmsnorm(y) * weight: the norm on a sublayer's output (post-norm blocks).  `cast`, if
-        given, receives the new stream in the compute type."""
-        ops.post_rmsnorm_add(residual, y, self.weight, self.eps, cast=cast)
+    def add_normed(self, residual, y, cast=None, next_norm=None):
+        """residual (float32) += rmsnorm(y) * weight: the norm on a sublayer's output.  `cast`, if given, receives the new
+        stream in the compute type, with next_norm (one that declares folds_into_products) already normed by it."""
+        if next_norm is None:
+            ops.post_rmsnorm_add(residual, y, self.weight, self.eps, cast=cast)
+        else:
+            ops.post_rmsnorm_add(residual, y, self.weight, self.eps, cast=cast, next_weight=next_norm.scale_weight(), next_eps=next_norm.eps)
 
 
 register_part("norm", "rmsnorm", RMSNorm)

@@ -83,7 +83,8 @@ class AttentionSpec:
 
 @dataclass(frozen=True)
 class SwiGLUSpec:
-    """Dense gated feed-forward: down(act(gate x) * up x); act 'silu' or 'gelu_tanh' (the tanh form of GELU)."""
+    """Dense gated feed-forward: down(act(gate x) * up x); act 'silu' or 'gelu_tanh' (the tanh form of GELU), or 'clamped':
+    g = min(gate x, limit), u = up x clamped to +-limit, down(g * sigmoid(slope * g) * (u + 1))."""
     hidden_size: int
     intermediate_size: int
     gate_proj: str
@@ -91,6 +92,8 @@ class SwiGLUSpec:
     down_proj: str
     kind: str = "swiglu"
     activation: str = "silu"
+    limit: float = 0.0            # of 'clamped'
+    slope: float = 0.0
 
     def tensors(self) -> TensorTable:
         return {self.gate_proj: ((self.intermediate_size, self.hidden_size), "matrix"),
@@ -239,7 +242,10 @@ class Mamba2Spec:
 class MoESpec:
     """Routed feed-forward: `experts` gated feed-forwards of which each token uses `top`, weighted by the
     softmax over the chosen router logits; optionally a shared gated feed-forward for every token, scaled
-    by the sigmoid of one number per token."""
+    by the sigmoid of one number per token (shared_gate) or added as it is.
+    With `correction` (a number per row of the router) scores are the softmax over ALL router logits, the choice goes by
+    score + correction and the weights are the chosen scores times route_scale.  The last `identity` rows of the router are
+    identity experts: their output is the input itself, they have no matrices."""
     hidden_size: int
     experts: int
     top: int
@@ -249,13 +255,21 @@ class MoESpec:
     shared: Optional[SwiGLUSpec] = None
     shared_gate: Optional[str] = None
     kind: str = "moe"
+    identity: int = 0
+    correction: Optional[str] = None
+    route_scale: float = 1.0      # with `correction`
+    activation: str = "silu"      # of the experts, as SwiGLUSpec's
+    limit: float = 0.0
+    slope: float = 0.0
 
     def expert_names(self, e: int):
         p = f"{self.expert_prefix}{e}."
         return p + "gate", p + "up", p + "down"
 
     def tensors(self) -> TensorTable:
-        t: TensorTable = {self.router: ((self.experts, self.hidden_size), "matrix")}
+        t: TensorTable = {self.router: ((self.experts + self.identity, self.hidden_size), "matrix")}
+        if self.correction is not None:
+            t[self.correction] = ((self.experts + self.identity,), "normal:0:0.01")
         for e in range(self.experts):
             g, u, dn = self.expert_names(e)
             t[g] = ((self.expert_ff, self.hidden_size), "matrix")
@@ -263,7 +277,8 @@ class MoESpec:
             t[dn] = ((self.hidden_size, self.expert_ff), "matrix")
         if self.shared is not None:
             t.update(self.shared.tensors())
-            t[self.shared_gate] = ((1, self.hidden_size), "matrix")
+            if self.shared_gate is not None:
+                t[self.shared_gate] = ((1, self.hidden_size), "matrix")
         return t
 
 
@@ -553,6 +568,81 @@ class RotNormAttentionSpec:
 
 
 @dataclass(frozen=True)
+class TalkingAttentionSpec:
+    """Causal grouped-query attention whose heads' softmax weights are mixed before they meet the values.  Queries and keys are
+    rotated over their first rotary_dim entries (`position`, a RotarySpec of either pairing, or None); the score is (q . k) * scale,
+    then softcap * tanh(score / softcap) where softcap > 0; head h's softmax has exp(sink[h]) in its denominator too; head h
+    applies sum_g talk[h, g] * (head g's weights) to the values of its own key/value head.  Key and value sizes are unrelated;
+    values may be shared between layers as for RotNormAttentionSpec."""
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    value_dim: int
+    scale: float
+    softcap: float                # 0: none
+    q_proj: str
+    k_proj: str
+    v_proj: str
+    o_proj: str
+    sink: str                     # [heads]
+    talk: str                     # [heads, heads]
+    position: Optional[object] = None
+    v_share: Optional[str] = None
+    v_share_role: Optional[str] = None        # 'source' | 'blend' | None
+    v_blend: Optional[str] = None             # a number; stored in every sharing layer, used by 'blend' layers
+    kind: str = "talking_attention"
+
+    def tensors(self) -> TensorTable:
+        H, G, n, dv, d = self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, self.hidden_size
+        t: TensorTable = {self.q_proj: ((H * n, d), "matrix"), self.k_proj: ((G * n, d), "matrix"), self.v_proj: ((G * dv, d), "matrix"),
+                          self.o_proj: ((d, H * dv), "matrix"), self.sink: ((H,), "normal:0:1"), self.talk: ((H, H), "normal:0.2:0.4")}
+        if self.v_blend is not None:
+            t[self.v_blend] = ((), "normal:0.4:0.1")
+        if self.position is not None:
+            t.update(self.position.tensors())
+        return t
+
+
+@dataclass(frozen=True)
+class HeadDeltaSpec:
+    """Delta rule with one decay per head whose removal reads the decayed state.  Per head (head h reads query/key group
+    h // (heads / kv_heads)): S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q.  q, k, v pass a short causal convolution per
+    channel (<name>.conv, [channels, taps], the current token's tap last) and SiLU; q and k are then unit vectors per head (key_eps
+    under the root), q times key_dim^(-1/2); beta = sigmoid(W_b x); g = exp(-exp(a_log) softplus(W_a x + dt_bias)) per head; o is
+    divided by its root mean square per head, weighted (norm, [value_dim], shared by the heads) and multiplied by silu(W_g x)."""
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    key_dim: int
+    value_dim: int
+    conv_taps: int
+    eps: float
+    q_proj: str
+    k_proj: str
+    v_proj: str
+    gate_proj: str
+    beta_proj: str
+    a_proj: str
+    dt_bias: str
+    a_log: str
+    norm: str
+    o_proj: str
+    key_eps: float = 1e-6
+    kind: str = "head_delta"
+
+    def tensors(self) -> TensorTable:
+        H, G, dk, dv, d = self.num_heads, self.num_kv_heads, self.key_dim, self.value_dim, self.hidden_size
+        t: TensorTable = {self.q_proj: ((G * dk, d), "matrix"), self.k_proj: ((G * dk, d), "matrix"), self.v_proj: ((H * dv, d), "matrix"),
+                          self.gate_proj: ((H * dv, d), "matrix"), self.beta_proj: ((H, d), "matrix"), self.a_proj: ((H, d), "matrix"),
+                          self.dt_bias: ((H,), "normal:-1:1"), self.a_log: ((H,), "normal:-1:0.5"), self.norm: ((dv,), "norm"),
+                          self.o_proj: ((d, H * dv), "matrix")}
+        for name, ch in ((self.q_proj, G * dk), (self.k_proj, G * dk), (self.v_proj, H * dv)):
+            t[name + ".conv"] = ((ch, self.conv_taps), "normal:0:0.4")
+        return t
+
+
+@dataclass(frozen=True)
 class ChannelDeltaSpec:
     """Delta rule with a decay per head and key channel whose removal reads the decayed state.  Per head (head h reads
     query/key group h // (heads / kv_heads)): S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q.
@@ -652,7 +742,8 @@ class LayerSpec:
     'gated_pre_norm' is 'pre_norm' with each part's output multiplied by sigmoid(W h + b), h being the part's input:
     mixer_gate / ffn_gate name W [width, width], the bias is name + ".b".
     'post_norm': x += mixer_norm(mixer(x)); x += ffn_norm(feed_forward(x)): the parts read the stream itself and the norms
-    sit on their outputs."""
+    sit on their outputs.
+    'sandwich_norm': x += mixer_post_norm(mixer(mixer_norm(x))); x += ffn_post_norm(feed_forward(ffn_norm(x)))."""
     mixer: object
     feed_forward: object
     mixer_norm: object
@@ -663,10 +754,12 @@ class LayerSpec:
     residual_mult: float = 1.0
     mixer_gate: Optional[str] = None
     ffn_gate: Optional[str] = None
+    mixer_post_norm: object = None
+    ffn_post_norm: object = None
 
     def tensors(self) -> TensorTable:
         t: TensorTable = {}
-        for part in (self.mixer_norm, self.mixer, self.ffn_norm, self.feed_forward):
+        for part in (self.mixer_norm, self.mixer, self.mixer_post_norm, self.ffn_norm, self.feed_forward, self.ffn_post_norm):
             if part is not None:
                 t.update(part.tensors())
         width = getattr(self.mixer_norm, "size", None)
