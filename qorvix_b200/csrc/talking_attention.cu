@@ -501,13 +501,9 @@ __global__ void __launch_bounds__(256) talking_slice_kernel(TalkArgs a, TalkSlic
   load(0, k_lo);
   for (int kb = 0; kb < nkb; ++kb) {
     const int j0 = k_lo + kb * KB, st = stages > 1 ? kb & 1 : 0;
-    if (stages > 1 && kb + 1 < nkb) {
-      load(st ^ 1, j0 + KB);
-      ta_wait<1>();
-    } else {
-      ta_wait<0>();
-    }
-    __syncthreads();
+    ta_wait<0>();
+    __syncthreads();                                      // the block is there, and nobody reads the other stage any more
+    if (stages > 1 && kb + 1 < nkb) load(st ^ 1, j0 + KB);
     const bf16* tK = ring + st * stage_elems;
     const bf16* tV = tK + KB * L.KR;
     // scores: a unit is 16 keys of one key/value head; the rows of other heads are dropped

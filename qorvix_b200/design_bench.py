@@ -1,9 +1,9 @@
-"""Prefill and decode throughput of a Deganex, a Lotirax, a Tubazen or a Lugizen model at layer sizes that resemble real models, beside the
+"""Prefill and decode throughput of a Deganex, a Lotirax, a Tubazen, a Lugizen or a Nedasun model at layer sizes that resemble real models, beside the
 Llama decoder at equal width, depth and (active) feed-forward size, and the design's kernels alone with their roofline
 fractions beside the Llama kernels they correspond to.
 
-    python bench.py --design deganex|lotirax|tubazen|lugizen [--layers-per-kind 2] [--batch 8] [--ctx 1024] [--prefill-tokens 2048]
-    python -m qorvix_b200.design_bench [--design lotirax|tubazen|lugizen]
+    python bench.py --design deganex|lotirax|tubazen|lugizen|nedasun [--layers-per-kind 2] [--batch 8] [--ctx 1024] [--prefill-tokens 2048]
+    python -m qorvix_b200.design_bench [--design lotirax|tubazen|lugizen|nedasun]
 
 Random bfloat16 weights; timing with CUDA events after warm-up; kernels alone are timed in captured chains over
 buffers larger than L2 (kernel_bench.timed_chain).  Figures go out as one JSON line.
@@ -168,15 +168,16 @@ def scan_case(kind, seg_lens, peaks) -> dict:
     return kb._figures(us, nbytes, 4.0 * T * H * dk * dv, peaks)
 
 
-def experts_case(T, peaks) -> dict:
-    """Both products of the routed experts for T tokens (router and grouping included, shared expert excluded)."""
+def experts_case(T, peaks, identity=0) -> dict:
+    """Both products of the routed experts for T tokens (router and grouping included, shared expert excluded); identity > 0: the
+    router that scores all experts, with that many identity experts (whose choices take no product) and clamped activations."""
     E, top, ff, d = MOE["router"]["experts"], MOE["router"]["top"], MOE["expert"]["ff"], WIDTH
     wbytes = E * 3 * ff * d * 2
     copies = max(2, int(2.5 * kb.L2_BYTES // wbytes) + 1)
     wg = [ops.moe_pack_experts(torch.randn(E, ff, d, device="cuda", dtype=torch.bfloat16) * 0.02) for _ in range(copies)]
     wu = [ops.moe_pack_experts(torch.randn(E, ff, d, device="cuda", dtype=torch.bfloat16) * 0.02) for _ in range(copies)]
     wd = [ops.moe_pack_experts(torch.randn(E, d, ff, device="cuda", dtype=torch.bfloat16) * 0.02) for _ in range(copies)]
-    router = torch.randn(E, d, device="cuda", dtype=torch.bfloat16)
+    router = torch.randn(E + identity, d, device="cuda", dtype=torch.bfloat16)
     x = torch.randn(T, d, device="cuda", dtype=torch.bfloat16)
     R = T * top
     top_idx = torch.empty(T, top, device="cuda", dtype=torch.int32)
@@ -187,15 +188,19 @@ def experts_case(T, peaks) -> dict:
     act = torch.empty(R, ff, device="cuda", dtype=torch.bfloat16)
     y = torch.empty(R, d, device="cuda", dtype=torch.float32)
     delta = torch.empty(T, d, device="cuda", dtype=torch.float32)
+    corr = torch.zeros(E + identity, device="cuda") if identity else None
+    glu = dict(act=ops.GLU_CLAMPED, limit=7.0, slope=1.702) if identity else {}
 
     def run(i):
-        ops.moe_route(top_idx, top_w, None, x, router, None)
+        ops.moe_route(top_idx, top_w, None, x, router, None, correction=corr, w_scale=2.5)
         ops.moe_group(row_token, slot_row, tiles, top_idx, scratch, E, tile_rows)
-        ops.moe_experts_tc(True, act, x, wg[i % copies], wu[i % copies], row_token, tiles)
+        ops.moe_experts_tc(True, act, x, wg[i % copies], wu[i % copies], row_token, tiles, **glu)
         ops.moe_experts_tc(False, y, act, wd[i % copies], None, row_token, tiles)
-        ops.moe_combine(delta, None, y, slot_row, top_w, None, None)
+        ops.moe_combine(delta, None, y, slot_row, top_w, None, None, identity_in=x if identity else None)
 
     us = kb.timed_chain(run, launches=6)
+    if identity:
+        R = int((top_idx < E).sum())                           # the choices that take a product
     touched = min(E, R)                                        # experts whose weights a step must read at least
     nbytes = touched * 3 * ff * d * 2 + T * d * 2 + R * (ff * 2 * 2 + d * 4 * 2) + T * d * 4
     return kb._figures(us, nbytes, 2.0 * R * 3 * ff * d, peaks)
@@ -640,6 +645,194 @@ def run_lugizen(args, peaks) -> dict:
     return res
 
 
+# ------------------------------------------------------------------ Nedasun
+# Attention of 16 heads of 128 on 4 key/value heads with soft-capped scores, sinks and mixed heads, values blended between layers; a
+# delta rule of 16 value heads of 128 on 8 query/key heads of 128 with one decay a head and convolutions of four taps; 64 experts of
+# 1,408 and 4 identity experts of which 6 serve a token beside a shared one of 2,816, or a dense feed-forward of the same active
+# size.  The recurrent layers and the attention layers are sized as Lugizen's.
+NED_ATTN = {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0, "rot": {"base": 10000.0, "dims": 128},
+            "v_mix": True}
+NED_DELTA = {"heads": 16, "kv_heads": 8, "dim": 128, "vdim": 128, "conv": 4}
+NED_MOE = {"kind": "moe", "expert": {"ff": 1408, "limit": 7.0}, "router": {"experts": 64, "identity": 4, "scale": 2.5, "top": 6},
+           "shared": {"ff": 2816, "limit": 7.0}}
+NED_DENSE = {"kind": "dense", "ff": 6 * 1408 + 2816, "limit": 7.0}
+
+
+def nedasun_config(layers_per_kind: int) -> dict:
+    """Pairs of a recurrent and an attention layer; the first pair's feed-forwards are dense, the others' routed."""
+    layers = []
+    for i in range(layers_per_kind):
+        f = NED_DENSE if i == 0 else NED_MOE
+        layers += [{"type": "delta", "mixer": NED_DELTA, "mlp": f}, {"type": "attention", "mixer": NED_ATTN, "mlp": f}]
+    return {"architecture": "Nedasun", "vocab": VOCAB, "width": WIDTH, "norm": {"eps": 1e-5}, "layers": layers}
+
+
+def nedasun_lugizen_config(layers_per_kind: int) -> dict:
+    """The closest model's layers in the same order and with the same feed-forward sizes (it has no shared expert)."""
+    layers = []
+    for i in range(layers_per_kind):
+        f = {"kind": "dense", "ff": NED_DENSE["ff"]} if i == 0 else LUG_MOE
+        layers += [{"type": "channel_delta", "mixer": LUG_DELTA, "mlp": f}, {"type": "attention", "mixer": LUG_ATTN, "mlp": f}]
+    return {"architecture": "Lugizen", "vocab": VOCAB, "width": WIDTH, "norm": {"eps": 1e-5}, "canon": {"taps": 4}, "layers": layers}
+
+
+def nedasun_llama_config(n_layers: int) -> dict:
+    return {"architectures": ["LlamaForCausalLM"], "vocab_size": VOCAB, "hidden_size": WIDTH, "intermediate_size": NED_DENSE["ff"],
+            "num_hidden_layers": n_layers, "num_attention_heads": 16, "num_key_value_heads": 4, "head_dim": 128,
+            "max_position_embeddings": 8192, "rms_norm_eps": 1e-5, "rope_theta": 10000.0, "tie_word_embeddings": False}
+
+
+def talking_attention_case(seg_lens, ctx_len, peaks, page=16) -> dict:
+    """Attention with mixed heads over the given segments, each ending at ctx_len cached tokens (the preparing kernel excluded)."""
+    a = NED_ATTN
+    H, G, n, dv = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+    S, T = len(seg_lens), sum(seg_lens)
+    blocks = -(-ctx_len // page)
+    width = G * (n + dv)
+    copies = max(2, min(8, int(2.5 * kb.L2_BYTES // (S * ctx_len * width * 2)) + 1))
+    caches = torch.randn(copies, S * blocks + 1, page, width, device="cuda", dtype=torch.bfloat16)
+    table = torch.arange(S * blocks, dtype=torch.int32, device="cuda").view(S, blocks)
+    ctx = _ctx(seg_lens, [ctx_len - m for m in seg_lens])
+    ctx.seg_len, ctx.seg_start_pos, ctx.max_ctx_len, ctx.captured = list(seg_lens), [ctx_len - m for m in seg_lens], ctx_len, False
+    ctx.seg_pos0 = torch.tensor(ctx.seg_start_pos, dtype=torch.int32, device="cuda")
+    q = torch.randn(T, H * n, device="cuda", dtype=torch.bfloat16)
+    out = torch.empty(T, H * dv, device="cuda", dtype=torch.bfloat16)
+    sink = torch.randn(H, device="cuda")
+    talk = torch.eye(H) + torch.randn(H, H) * 0.2
+    talk_dev = talk.cuda()
+    us = kb.timed_chain(lambda i: ops.talking_attention(out, q, caches[i % copies], ctx, table, H, G, n, dv, page, a["scale"], a["softcap"], sink,
+                                                        talk_dev, talk), launches=8)
+    pairs = sum(m * (ctx_len - m) + m * (m + 1) // 2 for m in seg_lens)
+    # a (query, key) pair: H products of n and of dv entries, and the mixing of H weights into H
+    return kb._figures(us, S * ctx_len * width * 2 + (q.numel() + out.numel()) * 2, pairs * H * (2.0 * n + 2.0 * dv + 2.0 * H), peaks)
+
+
+def talking_prepare_case(T, peaks, page=16) -> dict:
+    """Rotation in neighbouring pairs, blended values and the cache write of T tokens of one request."""
+    a = NED_ATTN
+    H, G, n, dv, rot = a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["rot"]["dims"]
+    cols, width = (H + G) * n + G * dv, G * (n + dv)
+    copies = max(2, min(8, int(2.5 * kb.L2_BYTES // (T * (cols * 4 + G * dv * 4 + width * 2 + H * n * 2))) + 1))
+    projs = torch.randn(copies, T, cols, device="cuda", dtype=torch.float32)
+    firsts = torch.randn(copies, T, G * dv, device="cuda", dtype=torch.float32)
+    blocks = -(-T // page)
+    caches = torch.zeros(copies, blocks + 1, page, width, device="cuda", dtype=torch.bfloat16)
+    table = torch.arange(blocks, dtype=torch.int32, device="cuda").view(1, blocks)
+    ctx = _ctx([T], [0])
+    ang = torch.arange(T, device="cuda", dtype=torch.float32)[:, None] * torch.rand(rot // 2, device="cuda")[None, :]
+    cos_sin = torch.stack([torch.cos(ang), torch.sin(ang)], dim=-1).contiguous()
+    q = torch.empty(copies, T, H * n, device="cuda", dtype=torch.bfloat16)
+    us = kb.timed_chain(lambda i: ops.rot_norm_prepare(q[i % copies], projs[i % copies], 0, H * n, (H + G) * n, caches[i % copies], cos_sin, rot, False,
+                                                       0.0, None, firsts[i % copies], 0.4, ctx, table, H, G, n, dv, page, interleaved=True), launches=8)
+    return kb._figures(us, T * (cols * 4 + G * dv * 4 + width * 2 + H * n * 2), 0.0, peaks)
+
+
+def head_delta_case(seg_lens, peaks, scan_only=False) -> dict:
+    """The delta rule with one decay a head: its chain (convolutions with SiLU, operands, recurrence, norm and gate), or (scan_only)
+    the recurrence's kernel alone."""
+    m = NED_DELTA
+    H, G, dk, dv, taps = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+    S, T = len(seg_lens), sum(seg_lens)
+    ctx = _ctx(seg_lens, [0] * S)
+    C = 2 * G * dk + H * dv
+    block = ops.head_delta_block(torch.bfloat16)
+    n_state = ops.head_delta_state_floats(H, dk, dv)
+    copies = max(2, min(8, int(2.5 * kb.L2_BYTES // (S * n_state * 4)) + 1))
+    states = torch.zeros(copies, S, n_state, device="cuda", dtype=torch.float32)
+    tails = torch.zeros(S, (taps - 1) * C, device="cuda", dtype=torch.float32)
+    f32 = dict(device="cuda", dtype=torch.float32)
+    proj = torch.randn(T, C + H * dv + 2 * H, **f32) * 0.3
+    conv_w = torch.randn(C, taps, **f32) * 0.3
+    dt_bias, rate, nw = torch.randn(H, **f32) - 2, torch.rand(H, **f32), torch.ones(H * dv, **f32)
+    conv, qn, kn = torch.empty(T, C, **f32), torch.empty(T, G * dk, **f32), torch.empty(T, G * dk, **f32)
+    coef, y = torch.empty(T, H, ops.head_delta_coef(), **f32), torch.empty(T, H * dv, **f32)
+    out = torch.empty(T, H * dv, device="cuda", dtype=torch.bfloat16)
+    g0 = C
+    b0 = g0 + H * dv
+
+    def prepare():
+        ops.conv_state(conv, proj[:, :C], conv_w, None, tails, ctx, act=True)
+        ops.head_delta_operands(qn, kn, coef, conv[:, : G * dk], conv[:, G * dk: 2 * G * dk], proj[:, b0 + H:], proj[:, b0: b0 + H], rate, dt_bias, ctx,
+                                H, G, dk, 1e-6, dk ** -0.5, block)
+    prepare()
+
+    def run(i):
+        if not scan_only:
+            prepare()
+        ops.head_delta_scan(y, qn, kn, conv[:, 2 * G * dk:], coef, states[i % copies], ctx, H, G, dk, dv, block)
+        if not scan_only:
+            ops.head_norm_gate(out, y, proj[:, g0:b0], nw, H, 1e-5, ops.HEAD_GATE_SILU)
+
+    us = kb.timed_chain(run, launches=6)
+    nbytes = 2 * S * n_state * 4 + T * (2 * G * dk + 2 * H * dv + H * ops.head_delta_coef()) * 4
+    if not scan_only:
+        nbytes += T * ((C + H * dv + 2 * H) * 4 + H * dv * 2)
+    return kb._figures(us, nbytes, 8.0 * T * H * dk * dv, peaks)
+
+
+def sandwich_norm_case(T, peaks) -> dict:
+    """A sublayer's output normed and added to the stream, and the next sublayer's input normed, in one pass."""
+    d = WIDTH
+    copies = max(2, min(8, int(2.5 * kb.L2_BYTES // (T * d * 12)) + 1))
+    res = torch.randn(copies, T, d, device="cuda", dtype=torch.float32)
+    y = torch.randn(copies, T, d, device="cuda", dtype=torch.bfloat16)
+    h = torch.empty(copies, T, d, device="cuda", dtype=torch.bfloat16)
+    g = torch.ones(d, device="cuda", dtype=torch.float32)
+    us = kb.timed_chain(lambda i: ops.post_rmsnorm_add(res[i % copies], y[i % copies], g, 1e-5, cast=h[i % copies], next_weight=g, next_eps=1e-5), launches=8)
+    return kb._figures(us, T * d * 12, 0.0, peaks)
+
+
+def clamped_gate_up_case(T, peaks, act) -> dict:
+    """The gate/up product with its activation in the epilogue (the clamped one, or SiLU for comparison)."""
+    ff, d = NED_DENSE["ff"], WIDTH
+    copies = max(2, int(2.5 * kb.L2_BYTES // (2 * ff * d * 2)) + 1)
+    ws = [ops.pack_weight(torch.randn(2 * ff, d, device="cuda", dtype=torch.bfloat16) * 0.02) for _ in range(copies)]
+    x = torch.randn(T, d, device="cuda", dtype=torch.bfloat16)
+    out = torch.empty(T, ff, device="cuda", dtype=torch.bfloat16)
+    us = kb.timed_chain(lambda i: ops.gemm_swiglu(out, x, None, ws[i % copies], 2 * ff, act=act, limit=7.0, slope=1.702), launches=8)
+    return kb._figures(us, 2 * ff * d * 2 + T * (d + ff) * 2, 2.0 * T * 2 * ff * d, peaks)
+
+
+def run_nedasun(args, peaks) -> dict:
+    n_layers = 2 * args.layers_per_kind
+    sizes = (args.batch, args.ctx, args.prefill_tokens, args.steps, args.warmup)
+    T, B, C = args.prefill_tokens, args.batch, args.ctx
+    res = {"nedasun": model_throughput(nedasun_config(args.layers_per_kind), *sizes),
+           "lugizen_equal_size": model_throughput(nedasun_lugizen_config(args.layers_per_kind), *sizes),
+           "llama_equal_size": model_throughput(nedasun_llama_config(n_layers), *sizes)}
+    res["kernels"] = {
+        f"talking_attention_prefill_t{T}": talking_attention_case([T], T, peaks),
+        f"talking_attention_prefill_t{T // 4}_ctx{T}": talking_attention_case([T // 4], T, peaks),
+        f"talking_attention_decode_b{B}_ctx{C}": talking_attention_case([1] * B, C, peaks),
+        f"talking_attention_decode_b{8 * B}_ctx{C}": talking_attention_case([1] * (8 * B), C, peaks),
+        f"talking_prepare_t{T}": talking_prepare_case(T, peaks), f"talking_prepare_t{B}": talking_prepare_case(B, peaks),
+        f"head_delta_prefill_t{T}": head_delta_case([T], peaks), f"head_delta_decode_b{B}": head_delta_case([1] * B, peaks),
+        f"head_delta_scan_alone_prefill_t{T}": head_delta_case([T], peaks, True), f"head_delta_scan_alone_decode_b{B}": head_delta_case([1] * B, peaks, True),
+        f"experts_prefill_t{T}": experts_case(T, peaks, identity=4), f"experts_decode_b{B}": experts_case(B, peaks, identity=4),
+        f"sandwich_norm_t{T}": sandwich_norm_case(T, peaks), f"sandwich_norm_t{B}": sandwich_norm_case(B, peaks),
+        f"clamped_gate_up_t{T}": clamped_gate_up_case(T, peaks, ops.GLU_CLAMPED), f"clamped_gate_up_t{B}": clamped_gate_up_case(B, peaks, ops.GLU_CLAMPED),
+    }
+    # the like kernels of the closest design at the same sizes: Lugizen's attention, its preparing kernel, its delta rule, the experts
+    # without identity experts, the norm on a sublayer's output and the pre-norm decoders' norm pass, the SiLU epilogue
+    res["like_kernels"] = {
+        f"attention_prefill_t{T}": plain_attention_case([T], T, peaks), f"attention_prefill_t{T // 4}_ctx{T}": plain_attention_case([T // 4], T, peaks),
+        f"attention_decode_b{B}_ctx{C}": plain_attention_case([1] * B, C, peaks), f"attention_decode_b{8 * B}_ctx{C}": plain_attention_case([1] * (8 * B), C, peaks),
+        f"rot_norm_prepare_t{T}": rot_norm_prepare_case(T, peaks), f"rot_norm_prepare_t{B}": rot_norm_prepare_case(B, peaks),
+        f"channel_delta_prefill_t{T}": channel_delta_case([T], peaks), f"channel_delta_decode_b{B}": channel_delta_case([1] * B, peaks),
+        f"channel_delta_scan_alone_prefill_t{T}": channel_delta_case([T], peaks, True),
+        f"channel_delta_scan_alone_decode_b{B}": channel_delta_case([1] * B, peaks, True),
+        f"experts_prefill_t{T}": experts_case(T, peaks), f"experts_decode_b{B}": experts_case(B, peaks),
+        f"norm_on_output_t{T}": stream_passes_case(T, peaks)["norm_on_output"], f"norm_on_output_t{B}": stream_passes_case(B, peaks)["norm_on_output"],
+        f"add_rmsnorm_t{T}": add_rmsnorm_case(T, peaks), f"add_rmsnorm_t{B}": add_rmsnorm_case(B, peaks),
+        f"silu_gate_up_t{T}": clamped_gate_up_case(T, peaks, ops.GLU_SILU), f"silu_gate_up_t{B}": clamped_gate_up_case(B, peaks, ops.GLU_SILU),
+    }
+    from .config import LlamaConfig
+    like = kb.headline_kernels(LlamaConfig.from_dict(nedasun_llama_config(n_layers)), B, C, T, peaks)
+    ops.check_kernel_errors()
+    res["llama_kernels"] = {k: v for k, v in like.items() if "attention" in k or "gate_up" in k or "down" in k}
+    return res
+
+
 def run(args, peaks) -> dict:
     n_layers = 3 * args.layers_per_kind
     res = {"deganex": model_throughput(deganex_config(args.layers_per_kind), args.batch, args.ctx, args.prefill_tokens, args.steps, args.warmup),
@@ -663,7 +856,7 @@ def run(args, peaks) -> dict:
 def main(argv=None, peaks=None, extra=None) -> int:
     """extra: a callable whose dict (the clocks sampled during the run, for instance) joins the JSON line."""
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("--design", default="deganex", choices=["deganex", "lotirax", "tubazen", "lugizen"])
+    ap.add_argument("--design", default="deganex", choices=["deganex", "lotirax", "tubazen", "lugizen", "nedasun"])
     ap.add_argument("--layers-per-kind", type=int, default=2)
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--ctx", type=int, default=1024)
@@ -678,6 +871,8 @@ def main(argv=None, peaks=None, extra=None) -> int:
         res, model = run_tubazen(args, peaks), f"Tubazen, width {WIDTH}, {2 * args.layers_per_kind} layers"
     elif args.design == "lugizen":
         res, model = run_lugizen(args, peaks), f"Lugizen, width {WIDTH}, {3 * args.layers_per_kind} layers"
+    elif args.design == "nedasun":
+        res, model = run_nedasun(args, peaks), f"Nedasun, width {WIDTH}, {2 * args.layers_per_kind} layers"
     else:
         res, model = run(args, peaks), f"Deganex, width {WIDTH}, {3 * args.layers_per_kind} layers"
     d = res[args.design]

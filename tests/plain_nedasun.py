@@ -65,18 +65,14 @@ def talking_attention(q, k, v, scale, cap, sink, talk):
     """q [T, H, n], k [T, G, n], v [T, G, dv]; causal.  Scores are soft-capped (cap None: not), every head's weights are
     softmaxed with its sink, then the weights of all heads are mixed (talk [H, H]) before they meet the values."""
     T, H, _ = q.shape
-    G = k.shape[1]
+    k, v = (x.repeat_interleave(H // x.shape[1], dim=1) for x in (k, v))              # every head's own key/value head
     out = torch.zeros(T, H, v.shape[2], dtype=F64)
     for i in range(T):
-        w = []
-        for h in range(H):
-            s = (k[: i + 1, h // (H // G)] @ q[i, h]) * scale
-            if cap:
-                s = cap * torch.tanh(s / cap)
-            w.append(sink_weights(s, sink[h]))
-        mixed = talk @ torch.stack(w)                                   # [H, i + 1]
-        for h in range(H):
-            out[i, h] = mixed[h] @ v[: i + 1, h // (H // G)]
+        s = torch.einsum("hn,jhn->hj", q[i], k[: i + 1]) * scale
+        if cap:
+            s = cap * torch.tanh(s / cap)
+        w = torch.stack([sink_weights(s[h], sink[h]) for h in range(H)])
+        out[i] = torch.einsum("hj,jhv->hv", talk @ w, v[: i + 1])
     return out
 
 
@@ -114,15 +110,13 @@ def gated_delta(h, W, p, m, eps, state=None):
     k = k / torch.sqrt((k * k).sum(-1, keepdim=True) + KEY_EPS)
     beta = torch.sigmoid(h @ W[p + "b"].T)                                                  # [T, H]
     g = torch.exp(-torch.exp(W[p + "A_log"]) * torch.nn.functional.softplus(h @ W[p + "a"].T + W[p + "dt_bias"]))
+    q, k = q.repeat_interleave(H // G, dim=1), k.repeat_interleave(H // G, dim=1)      # every head's own query/key head
     o = torch.zeros(T, H, dv, dtype=F64)
-    S = S.clone()
     for t in range(T):
-        for hd in range(H):
-            c = hd // (H // G)
-            S[hd] = g[t, hd] * S[hd]
-            u = beta[t, hd] * (v[t, hd] - S[hd].T @ k[t, c])
-            S[hd] = S[hd] + torch.outer(k[t, c], u)
-            o[t, hd] = S[hd].T @ q[t, c]
+        S = g[t][:, None, None] * S
+        u = beta[t][:, None] * (v[t] - torch.einsum("hnv,hn->hv", S, k[t]))
+        S = S + torch.einsum("hn,hv->hnv", k[t], u)
+        o[t] = torch.einsum("hnv,hn->hv", S, q[t])
     o = unit(o, eps) * W[p + "norm"] * silu(h @ W[p + "g"].T).reshape(T, H, dv)
     return o.reshape(T, H * dv) @ W[p + "o"].T, (S, new_tails)
 
@@ -133,13 +127,22 @@ def clamped_ff(h, W, p, limit):
     return (g * torch.sigmoid(SLOPE * g) * (u + 1.0)) @ W[p + "down"].T
 
 
-def routed_ff(h, W, p, f):
+def routed_ff(h, W, p, f, clear=None):
     """Softmax over all experts (those that only pass their input on included); chosen by score + correction; weighted by the
-    score times a fixed factor."""
+    score times a fixed factor.  clear, if a list, receives for every token whether its choice is no close call: the last
+    chosen and the first left out do not change places if either's router logit moves by 8 % of the logits' size."""
     r = f["router"]
     E, ident, top = r["experts"], r.get("identity", 0), r["top"]
-    s = torch.softmax(h @ W[p + "router"].T, dim=-1)
+    z = h @ W[p + "router"].T
+    s = torch.softmax(z, dim=-1)
     assert s.shape[1] == E + ident
+    if clear is not None:
+        if top < E + ident:
+            ranked, order = torch.sort(s + W[p + "correction"], dim=-1, descending=True)
+            moves = (s * (1 - s)).gather(1, order)[:, top - 1: top + 1].sum(dim=-1) * 0.08 * z.pow(2).mean(dim=-1).sqrt()
+            clear.append(ranked[:, top - 1] - ranked[:, top] > moves)
+        else:
+            clear.append(torch.ones(h.shape[0], dtype=torch.bool))
     out = torch.zeros_like(h)
     for t in range(h.shape[0]):
         for e in torch.topk(s[t] + W[p + "correction"], top).indices.tolist():
@@ -150,12 +153,12 @@ def routed_ff(h, W, p, f):
     return out
 
 
-def feed_forward(h, W, p, f):
-    return clamped_ff(h, W, p, f["limit"]) if f["kind"] == "dense" else routed_ff(h, W, p, f)
+def feed_forward(h, W, p, f, clear=None):
+    return clamped_ff(h, W, p, f["limit"]) if f["kind"] == "dense" else routed_ff(h, W, p, f, clear)
 
 
-def forward(cfg, W, tokens, taps=None):
-    """Logits [T, vocab] of one whole sequence; taps, if a list, receives the stream after every layer."""
+def forward(cfg, W, tokens, taps=None, clear=None):
+    """Logits [T, vocab] of one whole sequence; taps, if a list, receives the stream after every layer, clear as for routed_ff."""
     eps = float(cfg["norm"]["eps"])
     x = W["embed"][torch.as_tensor(tokens, dtype=torch.long)]
     v_first = None
@@ -175,7 +178,7 @@ def forward(cfg, W, tokens, taps=None):
         x = x + norm(y, W[p + "norm1b"], eps)
         f = layer.get("mlp")
         if f is not None:
-            y = feed_forward(norm(x, W[p + "norm2"], eps), W, p + "mlp.", f)
+            y = feed_forward(norm(x, W[p + "norm2"], eps), W, p + "mlp.", f, clear)
             x = x + norm(y, W[p + "norm2b"], eps)
         if taps is not None:
             taps.append(x.clone())
