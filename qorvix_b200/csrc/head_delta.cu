@@ -22,6 +22,7 @@
 // Everything is float32.  With block = 1 (what the 32-bit path uses, and what single tokens amount to in any case) the order of
 // every sum depends on the sizes alone; with block = 4 it also depends on where a portion starts, that is, cuts agree to rounding.
 #include "common.cuh"
+#include <type_traits>
 
 // factors per token and head: beta, beta G, G, g, then beta D(t, i) k_t.k_i for i < 3, then D(t, i) q_t.k_i for i < 4
 #define HD_COEF 12
@@ -209,6 +210,63 @@ __global__ void __launch_bounds__(32 * HD_WARPS) head_delta_scan_kernel(HeadDelt
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
+  // up to B tokens at a time (FULL: all B, without a branch, so that their reads and sums interleave)
+  auto tokens = [&](const float* d, int j, int nb, auto full) {
+    constexpr bool FULL = decltype(full)::value;
+    float p[B], r[B], u[B], e[B];
+#pragma unroll
+    for (int t = 0; t < B; ++t) {
+      p[t] = r[t] = 0.f;
+      if (FULL || t < nb) {
+        p[t] = hd_dot((const float4*)(d + t * ROW + lic * HD_PAD), S);
+        r[t] = hd_dot((const float4*)(d + t * ROW + VEC + lic * HD_PAD), S);
+      }
+    }
+#pragma unroll
+    for (int o = LPC / 2; o > 0; o >>= 1)
+#pragma unroll
+      for (int t = 0; t < B; ++t) {
+        p[t] += __shfl_xor_sync(0xffffffffu, p[t], o);
+        r[t] += __shfl_xor_sync(0xffffffffu, r[t], o);
+      }
+    float Gall = 1.0f;
+#pragma unroll
+    for (int t = 0; t < B; ++t) {
+      u[t] = 0.f;
+      e[t] = 1.f;
+      if (FULL || t < nb) {
+        const float* f = d + t * ROW + 2 * VEC;
+        const float4 f0 = *(const float4*)f, f1 = *(const float4*)(f + 4), f2 = *(const float4*)(f + 8);
+        const float kkc[3] = {f1.x, f1.y, f1.z}, qkc[4] = {f1.w, f2.x, f2.y, f2.z};
+        float uu = fmaf(f0.x, f[HD_COEF + warp * CPW + cw], -f0.y * p[t]);
+#pragma unroll
+        for (int i = 0; i < t; ++i) uu = fmaf(-kkc[i], u[i], uu);
+        u[t] = uu;
+        float y = f0.z * r[t];
+#pragma unroll
+        for (int i = 0; i <= t; ++i) y = fmaf(qkc[i], u[i], y);
+        if (lic == 0 && col < dv) a.out[(size_t)(q0 + j + t) * a.ld_out + hv + col] = y;
+        Gall = f0.z;
+#pragma unroll
+        for (int i = 0; i < t; ++i) e[i] *= f0.w;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < HD_ROWS; ++i) S[i] *= Gall;
+#pragma unroll
+    for (int t = 0; t < B; ++t) {
+      if (FULL || t < nb) {
+        const float ue = u[t] * e[t];
+        const float4* pk = (const float4*)(d + t * ROW + lic * HD_PAD);
+#pragma unroll
+        for (int i = 0; i < HD_ROWS / 4; ++i) {
+          const float4 k4 = pk[i];
+          S[4 * i] = fmaf(k4.x, ue, S[4 * i]); S[4 * i + 1] = fmaf(k4.y, ue, S[4 * i + 1]);
+          S[4 * i + 2] = fmaf(k4.z, ue, S[4 * i + 2]); S[4 * i + 3] = fmaf(k4.w, ue, S[4 * i + 3]);
+        }
+      }
+    }
+  };
   const int nchunks = (len + chunk - 1) / chunk;
   if (nchunks > 0) issue(0);
   for (int ch = 0; ch < nchunks; ++ch) {
@@ -221,63 +279,10 @@ __global__ void __launch_bounds__(32 * HD_WARPS) head_delta_scan_kernel(HeadDelt
     __syncthreads();
     const int j0 = ch * chunk, nt = min(chunk, len - j0);
     if (active) {
-      for (int jb = 0; jb < nt; jb += B) {
-        const float* d = hd_ring + ((size_t)(ch & 1) * chunk + jb) * ROW;
-        const int nb = min(B, nt - jb);
-        float p[B], r[B], u[B], e[B];
-#pragma unroll
-        for (int t = 0; t < B; ++t) {
-          p[t] = r[t] = 0.f;
-          if (t < nb) {
-            p[t] = hd_dot((const float4*)(d + t * ROW + lic * HD_PAD), S);
-            r[t] = hd_dot((const float4*)(d + t * ROW + VEC + lic * HD_PAD), S);
-          }
-        }
-#pragma unroll
-        for (int o = LPC / 2; o > 0; o >>= 1)
-#pragma unroll
-          for (int t = 0; t < B; ++t) {
-            p[t] += __shfl_xor_sync(0xffffffffu, p[t], o);
-            r[t] += __shfl_xor_sync(0xffffffffu, r[t], o);
-          }
-        float Gall = 1.0f;
-#pragma unroll
-        for (int t = 0; t < B; ++t) {
-          u[t] = 0.f;
-          e[t] = 1.f;
-          if (t < nb) {
-            const float* f = d + t * ROW + 2 * VEC;
-            const float4 f0 = *(const float4*)f, f1 = *(const float4*)(f + 4), f2 = *(const float4*)(f + 8);
-            const float kkc[3] = {f1.x, f1.y, f1.z}, qkc[4] = {f1.w, f2.x, f2.y, f2.z};
-            float uu = fmaf(f0.x, f[HD_COEF + warp * CPW + cw], -f0.y * p[t]);
-#pragma unroll
-            for (int i = 0; i < t; ++i) uu = fmaf(-kkc[i], u[i], uu);
-            u[t] = uu;
-            float y = f0.z * r[t];
-#pragma unroll
-            for (int i = 0; i <= t; ++i) y = fmaf(qkc[i], u[i], y);
-            if (lic == 0 && col < dv) a.out[(size_t)(q0 + j0 + jb + t) * a.ld_out + hv + col] = y;
-            Gall = f0.z;
-#pragma unroll
-            for (int i = 0; i < t; ++i) e[i] *= f0.w;
-          }
-        }
-#pragma unroll
-        for (int i = 0; i < HD_ROWS; ++i) S[i] *= Gall;
-#pragma unroll
-        for (int t = 0; t < B; ++t) {
-          if (t < nb) {
-            const float ue = u[t] * e[t];
-            const float4* pk = (const float4*)(d + t * ROW + lic * HD_PAD);
-#pragma unroll
-            for (int i = 0; i < HD_ROWS / 4; ++i) {
-              const float4 k4 = pk[i];
-              S[4 * i] = fmaf(k4.x, ue, S[4 * i]); S[4 * i + 1] = fmaf(k4.y, ue, S[4 * i + 1]);
-              S[4 * i + 2] = fmaf(k4.z, ue, S[4 * i + 2]); S[4 * i + 3] = fmaf(k4.w, ue, S[4 * i + 3]);
-            }
-          }
-        }
-      }
+      const float* d = hd_ring + (size_t)(ch & 1) * chunk * ROW;
+      int jb = 0;
+      for (; jb + B <= nt; jb += B) tokens(d + jb * ROW, j0 + jb, B, std::true_type{});
+      if (jb < nt) tokens(d + jb * ROW, j0 + jb, nt - jb, std::false_type{});
     }
     __syncthreads();
   }
@@ -324,8 +329,8 @@ extern "C" int qv_head_delta_scan(float* out, int ld_out, const float* qn, const
   dim3 grid(S, H, ctas), blk(32 * HD_WARPS);
   cudaStream_t st = (cudaStream_t)stream;
   const int row = 2 * HD_PAD * lpc + HD_COEF + cta_cols;
-  int chunk = max_q_len <= 1 ? 1 : (max_q_len > 16 ? 16 : (max_q_len + 3) / 4 * 4);
-  while (chunk > HD_BLOCK && (size_t)2 * chunk * row * sizeof(float) > 96 * 1024) chunk >>= 1;
+  int chunk = max_q_len <= 1 ? 1 : (max_q_len > 32 ? 32 : (max_q_len + 3) / 4 * 4);
+  while (chunk > HD_BLOCK && (size_t)2 * chunk * row * sizeof(float) > 96 * 1024) chunk -= HD_BLOCK;
   if (block > 1 && chunk < HD_BLOCK) chunk = HD_BLOCK;
   const size_t smem = (size_t)2 * chunk * row * sizeof(float);
   const int vec4 = dk % 4 == 0 && (((uintptr_t)qn | (uintptr_t)kn) & 15) == 0;

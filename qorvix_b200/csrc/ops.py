@@ -966,11 +966,13 @@ def talking_attention_slices(tokens: int, H: int, values: int, max_ctx: int):
     return max(1, -(-max_ctx // keys)), keys
 
 
-def talking_attention_cluster(tiles: int) -> int:
-    """CTAs that share out the keys of one tile of 16 tokens: few tiles are spread over more SMs."""
-    sms = sm_count()
+def talking_attention_cluster(seg_len, seg_pos0) -> int:
+    """CTAs that share out the keys of one tile of 16 tokens: as many as it takes for the longest tile not to outlast one and a
+    half times what the step's keys come to when every SM works."""
+    ends = [p + min(i + 16, m) for m, p in zip(seg_len, seg_pos0) for i in range(0, m, 16)]
+    longest, each = max(ends), sum(ends) / sm_count()
     c = 1
-    while c < 8 and tiles * c < 3 * sms // 2:
+    while c < 8 and longest > 1.5 * each * c:
         c *= 2
     return c
 
@@ -992,7 +994,7 @@ def talking_attention(out, q, cache_layer, ctx, block_table, H, G, n, dv, page, 
         if ok and n1 < S:
             lens = ctx.seg_len[n1:]
             ok = talking_attention_tc(out, q, cache_layer, ctx.seg_q_start[n1:], ctx.seg_pos0[n1:], block_table[n1:], S - n1, max(lens), *args,
-                                      cluster=talking_attention_cluster(sum(-(-m // 16) for m in lens)))
+                                      cluster=talking_attention_cluster(lens, ctx.seg_start_pos[n1:]))
         if ok:
             return
     talking_attention_generic(out, q, cache_layer, ctx, block_table, H, G, n, dv, page, scale, cap, sink, talk)

@@ -23,10 +23,13 @@
 //                  talking_merge_kernel joins the slices, divides and mixes.
 #include "common.cuh"
 #include <cooperative_groups.h>
+#include <type_traits>
 namespace cg = cooperative_groups;
 
 #define TA_KEYS 32
 #define TA_MAX_H 16                // heads of the tensor-core kernels
+#define TA_PS 36                   // row and head strides of the weights in shared memory (floats)
+#define TA_HS (16 * TA_PS + 4)
 #define TA_LOG2E 1.4426950408889634f
 
 // ---------------------------------------------------------------- float32 and other sizes
@@ -132,9 +135,10 @@ struct TalkArgs {
   float pre, post;                                 // score in base 2 = post * f(pre * dot): capped f = tanh, else the identity
   int capped;
   const float* sink;
+  const float* talk; int talk_terms;               // [H, H]; terms 1: every entry is a bfloat16 number, else 3
   float* partial; int slices; int slice_keys;      // single tokens: [S, slices, H, 2 + G * dv] (m, l, o)
 };
-// the mixing matrix rides in the kernel's parameters: its entries are then operands of the multiply-adds (no loads)
+// for few heads the mixing matrix rides in the kernel's parameters: its entries are then operands of the multiply-adds (no loads)
 template <int HP> struct TalkMatrix { float t[HP * HP]; };
 
 __device__ __forceinline__ void ta_ldsm4(uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3, const void* p) {
@@ -172,30 +176,41 @@ __device__ __forceinline__ void ta_split3(float x, float y, uint32_t& t0, uint32
   t1 = ta_pack(xr, yr);
   t2 = ta_pack(xr - __uint_as_float(t1 << 16), yr - __uint_as_float(t1 & 0xffff0000u));
 }
+// 2^x and 1 / x as the special-function unit gives them (two float32 ulp, one ulp; results below the smallest normal number are zero)
+__device__ __forceinline__ float ta_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float ta_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 // post * tanh(x) through one exponential: tanh(x) = 1 - 2 / (1 + e^(2x)); the error is an ulp of the cap
 __device__ __forceinline__ float ta_score(float dot, const TalkArgs& a) {
   const float x = dot * a.pre;
   if (!a.capped) return x;
-  return a.post - __fdividef(2.0f * a.post, 1.0f + exp2f(x));        // pre carries 2 log2 e here
+  return fmaf(-2.0f * a.post, ta_rcp(1.0f + ta_exp2(x)), a.post);    // pre carries 2 log2 e here
 }
 
 // ---- portions: 16 tokens, all heads
-// shared memory: sQ [H][16][KS], two buffers of [G][32][max(KS, VS)], sP [H][16][36] float, stats [2][H][16] float; the
+// shared memory: sQ [H][16][KS], two buffers of [G][32][max(KS, VS)], sP [H][TA_HS] float, stats [2][H][16] float; the
 // cluster's partial outputs [H][16][dv + 4] float lie over the front at the end
 static inline size_t ta_buf_bytes(int G, int NP, int DP) { return (size_t)G * TA_KEYS * ((NP > DP ? NP : DP) + 8) * sizeof(bf16); }
 static inline size_t ta_tile_smem(int H, int G, int NP, int DP, int dv) {
   const size_t front = (size_t)H * 16 * (NP + 8) * sizeof(bf16) + 2 * ta_buf_bytes(G, NP, DP);
-  const size_t body = front + (size_t)H * 16 * 36 * sizeof(float);
+  const size_t body = front + (size_t)H * TA_HS * sizeof(float);
   const size_t outs = (size_t)H * 16 * (dv + 4) * sizeof(float);
   return (body > outs ? body : outs) + (size_t)2 * H * 16 * sizeof(float);
 }
 
 template <int NP, int DP, int HP>
-__global__ void __launch_bounds__(HP * 32) talking_tile_kernel(TalkArgs a, const __grid_constant__ TalkMatrix<HP> mix, int cs, size_t stat_off) {
+__global__ void __launch_bounds__(HP * 32) talking_tile_kernel(TalkArgs a, const __grid_constant__ TalkMatrix<HP < 16 ? HP : 1> mix, int cs, size_t stat_off) {
   extern __shared__ __align__(16) unsigned char ta_smem[];
   constexpr int KS = NP + 8, VS = DP + 8;                 // row strides: an odd number of 16-byte units
   constexpr int KC = NP / 8, VC = DP / 8, BS = (NP > DP ? KS : VS);
-  constexpr int PS = 36;
+  constexpr int PS = TA_PS, HS = TA_HS;
   const int H = a.H, G = a.G, n = a.n, dv = a.dv, page = a.page, gs = H / G, NT = 32 * H;
   bf16* sQ = (bf16*)ta_smem;
   bf16* buf0 = sQ + H * 16 * KS;
@@ -218,22 +233,26 @@ __global__ void __launch_bounds__(HP * 32) talking_tile_kernel(TalkArgs a, const
     const bf16* src = valid ? a.q + (size_t)(q0 + rb * 16 + r) * a.ld_q + (size_t)hh * n + c * 8 : a.q;
     ta_cp16(sQ + hr * KS + c * 8, src, valid);
   }
-  // a block of keys (or values) of all key/value heads; lane r of every warp works out where key j0 + r lies
-  auto load = [&](bf16* dst, int j0, bool values) {
-    const int jr = j0 + lane;
+  // a block of keys (or values) of all key/value heads: a warp copies whole rows; lane r works out where key j0 + r lies
+  auto load = [&](bf16* dst, int j0, auto values) {
+    constexpr bool V = decltype(values)::value;
+    constexpr int C = V ? VC : KC, stride = V ? VS : KS;
+    const int jr = j0 + lane, size = V ? dv : n;
     unsigned long long row_at = 0;
-    if (jr < k_hi) row_at = ((unsigned long long)bt[jr / page] * page + (unsigned long long)(jr % page)) * width;
-    const int C = values ? VC : KC, size = values ? dv : n, stride = values ? VS : KS;
-    const size_t off = values ? (size_t)G * n : 0;
-    const int per = G * C;
-    for (int idx = tid; idx < TA_KEYS * per; idx += NT) {
-      const int r = idx / per, gc = idx - r * per, g = gc / C, c = gc - g * C;
-      const unsigned long long at = __shfl_sync(0xffffffffu, row_at, r);
-      const bool valid = j0 + r < k_hi && c * 8 < size;
-      ta_cp16(dst + (g * TA_KEYS + r) * stride + c * 8, valid ? a.cache + at + off + (size_t)g * size + c * 8 : a.cache, valid);
+    if (jr < k_hi) row_at = ((unsigned long long)bt[jr / page] * page + (unsigned long long)(jr % page)) * width + (V ? G * n : 0);
+    for (int r = h; r < TA_KEYS; r += H) {
+      const bf16* row = a.cache + __shfl_sync(0xffffffffu, row_at, r);
+      const bool in = j0 + r < k_hi;
+      for (int gc = lane; gc < G * C; gc += 32) {
+        const int g = gc / C, c = gc % C;
+        const bool valid = in && c * 8 < size;
+        ta_cp16(dst + (g * TA_KEYS + r) * stride + c * 8, valid ? row + g * size + c * 8 : a.cache, valid);
+      }
     }
     ta_commit();
   };
+  constexpr std::false_type KEYS{};
+  constexpr std::true_type VALUES{};
   const int pos_lo = min(i0 + g8, k_hi - 1), pos_hi = min(i0 + g8 + 8, k_hi - 1);
   const int mat = lane >> 3, r8 = lane & 7;
   // this head's scores of a block (base 2, capped, keys behind a row's position -inf)
@@ -269,10 +288,10 @@ __global__ void __launch_bounds__(HP * 32) talking_tile_kernel(TalkArgs a, const
   const float snk = a.sink[h] * TA_LOG2E;
   float m_lo = snk, m_hi = snk, l_lo = 0.f, l_hi = 0.f;   // finite from the start: a row may see nothing of a block
   // pass 1: maximum and sum (the sink's share is added once, below)
-  if (rank < nkb) load(buf0, rank * TA_KEYS, false);
+  if (rank < nkb) load(buf0, rank * TA_KEYS, KEYS);
   for (int kb = rank, it = 0; kb < nkb; kb += cs, ++it) {
     if (kb + cs < nkb) {
-      load((it & 1) ? buf0 : buf1, (kb + cs) * TA_KEYS, false);
+      load((it & 1) ? buf0 : buf1, (kb + cs) * TA_KEYS, KEYS);
       ta_wait<1>();
     } else {
       ta_wait<0>();
@@ -293,15 +312,15 @@ __global__ void __launch_bounds__(HP * 32) talking_tile_kernel(TalkArgs a, const
     float s_lo = 0.f, s_hi = 0.f;
 #pragma unroll
     for (int nt = 0; nt < 4; ++nt) {
-      s_lo += exp2f(sc[nt][0] - mx_lo) + exp2f(sc[nt][1] - mx_lo);
-      s_hi += exp2f(sc[nt][2] - mx_hi) + exp2f(sc[nt][3] - mx_hi);
+      s_lo += ta_exp2(sc[nt][0] - mx_lo) + ta_exp2(sc[nt][1] - mx_lo);
+      s_hi += ta_exp2(sc[nt][2] - mx_hi) + ta_exp2(sc[nt][3] - mx_hi);
     }
-    l_lo = l_lo * exp2f(m_lo - mx_lo) + s_lo;
-    l_hi = l_hi * exp2f(m_hi - mx_hi) + s_hi;
+    l_lo = l_lo * ta_exp2(m_lo - mx_lo) + s_lo;
+    l_hi = l_hi * ta_exp2(m_hi - mx_hi) + s_hi;
     m_lo = mx_lo; m_hi = mx_hi;
     __syncthreads();
   }
-  if (rank < nkb) load(buf0, rank * TA_KEYS, false);      // pass 2's first keys; flies while the sums are joined
+  if (rank < nkb) load(buf0, rank * TA_KEYS, KEYS);      // pass 2's first keys; flies while the sums are joined
   l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1); l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
   l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1); l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
   if (cs > 1) {
@@ -319,14 +338,27 @@ __global__ void __launch_bounds__(HP * 32) talking_tile_kernel(TalkArgs a, const
     float L_lo = 0.f, L_hi = 0.f;
     for (int r = 0; r < cs; ++r) {
       const float* o = cl.map_shared_rank(stat, r);
-      L_lo += o[(H + h) * 16 + g8] * exp2f(o[h * 16 + g8] - M_lo);
-      L_hi += o[(H + h) * 16 + g8 + 8] * exp2f(o[h * 16 + g8 + 8] - M_hi);
+      L_lo += o[(H + h) * 16 + g8] * ta_exp2(o[h * 16 + g8] - M_lo);
+      L_hi += o[(H + h) * 16 + g8 + 8] * ta_exp2(o[h * 16 + g8 + 8] - M_hi);
     }
     m_lo = M_lo; m_hi = M_hi; l_lo = L_lo; l_hi = L_hi;
   }
-  const float inv_lo = 1.0f / (l_lo + exp2f(snk - m_lo)), inv_hi = 1.0f / (l_hi + exp2f(snk - m_hi));
+  const float inv_lo = 1.0f / (l_lo + ta_exp2(snk - m_lo)), inv_hi = 1.0f / (l_hi + ta_exp2(snk - m_hi));
 
   // pass 2
+  // the mixing matrix as a product's first operand: its bfloat16 term `term` (0: rounded, 1: what is left rounded, 2: and again)
+  auto talk_operand = [&](int term, uint32_t (&tf)[4]) {
+#pragma unroll
+    for (int x = 0; x < 4; ++x) {
+      const int row = g8 + (x & 1) * 8, col = 2 * tg + (x >> 1) * 8;
+      const float t0 = row < H && col < H ? a.talk[row * H + col] : 0.f, t1 = row < H && col + 1 < H ? a.talk[row * H + col + 1] : 0.f;
+      uint32_t y[3];
+      ta_split3(t0, t1, y[0], y[1], y[2]);
+      tf[x] = term == 0 ? y[0] : term == 1 ? y[1] : y[2];
+    }
+  };
+  uint32_t tf[4];
+  if constexpr (HP == 16) talk_operand(0, tf);
   float o[DP / 8][4];
 #pragma unroll
   for (int i = 0; i < DP / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
@@ -334,37 +366,65 @@ __global__ void __launch_bounds__(HP * 32) talking_tile_kernel(TalkArgs a, const
     const int j0 = kb * TA_KEYS;
     ta_wait<0>();
     __syncthreads();                                      // the keys are there; values and weights of the last block are used up
-    load(buf1, j0, true);
+    load(buf1, j0, VALUES);
     {
       float sc[4][4];
       scores(buf0, j0, sc);
-      float* pw = sP + h * 16 * PS;
+      float* pw = sP + h * HS;
 #pragma unroll
       for (int nt = 0; nt < 4; ++nt) {
-        *(float2*)(pw + g8 * PS + nt * 8 + 2 * tg) = make_float2(exp2f(sc[nt][0] - m_lo) * inv_lo, exp2f(sc[nt][1] - m_lo) * inv_lo);
-        *(float2*)(pw + (g8 + 8) * PS + nt * 8 + 2 * tg) = make_float2(exp2f(sc[nt][2] - m_hi) * inv_hi, exp2f(sc[nt][3] - m_hi) * inv_hi);
+        *(float2*)(pw + g8 * PS + nt * 8 + 2 * tg) = make_float2(ta_exp2(sc[nt][0] - m_lo) * inv_lo, ta_exp2(sc[nt][1] - m_lo) * inv_lo);
+        *(float2*)(pw + (g8 + 8) * PS + nt * 8 + 2 * tg) = make_float2(ta_exp2(sc[nt][2] - m_hi) * inv_hi, ta_exp2(sc[nt][3] - m_hi) * inv_hi);
       }
     }
     __syncthreads();                                      // all heads' weights are there; the keys are used up
-    if (kb + cs < nkb) load(buf0, (kb + cs) * TA_KEYS, false);
+    if (kb + cs < nkb) load(buf0, (kb + cs) * TA_KEYS, KEYS);
     else ta_commit();                                     // an empty group, so that the counts below hold
+    if constexpr (HP == 16) {
+      // eight (query, key) pairs of one query a product: talk [16 x 16] times the heads' weights of the pairs (as three bfloat16
+      // terms), in place: the tile of pairs belongs to this warp
+      for (int tile = h; tile < 16 * TA_KEYS / 8; tile += H) {
+        float* pp = sP + (tile >> 2) * PS + (tile & 3) * 8;
+        uint32_t b[3][2];
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const int g = 2 * tg + 8 * x;
+          const float w0 = g < H ? pp[g * HS + g8] : 0.f, w1 = g + 1 < H ? pp[(g + 1) * HS + g8] : 0.f;
+          ta_split3(w0, w1, b[0][x], b[1][x], b[2][x]);
+        }
+        float c[4] = {0.f, 0.f, 0.f, 0.f};
+        if (a.talk_terms > 1) {                           // a matrix that bfloat16 does not hold exactly
+          uint32_t t1[4], t2[4];
+          talk_operand(1, t1);
+          talk_operand(2, t2);
+          ta_mma(c, t2, b[0][0], b[0][1]);
+          ta_mma(c, t1, b[1][0], b[1][1]);
+          ta_mma(c, t1, b[0][0], b[0][1]);
+        }
+#pragma unroll
+        for (int term = 2; term >= 0; --term) ta_mma(c, tf, b[term][0], b[term][1]);
+        __syncwarp();
+        if (g8 < H) *(float2*)(pp + g8 * HS + 2 * tg) = make_float2(c[0], c[1]);
+        if (g8 + 8 < H) *(float2*)(pp + (g8 + 8) * HS + 2 * tg) = make_float2(c[2], c[3]);
+      }
+    } else
     for (int pr = tid; pr < 16 * TA_KEYS; pr += NT) {     // one (query, key) a thread: all heads mixed in place
       float* pp = sP + (pr >> 5) * PS + (pr & 31);
       float p[HP];
 #pragma unroll
-      for (int g = 0; g < HP; ++g) p[g] = g < H ? pp[g * 16 * PS] : 0.f;
+      for (int g = 0; g < HP; ++g) p[g] = g < H ? pp[g * HS] : 0.f;
 #pragma unroll
       for (int hh = 0; hh < HP; ++hh) {
         float w = 0.f;
 #pragma unroll
-        for (int g = 0; g < HP; ++g) w = fmaf(mix.t[hh * HP + g], p[g], w);
-        if (hh < H) pp[hh * 16 * PS] = w;
+        for (int g = 0; g < HP; ++g) w = fmaf(mix.t[HP < 16 ? hh * HP + g : 0], p[g], w);
+        if (hh < H) pp[hh * HS] = w;
       }
     }
     ta_wait<1>();
     __syncthreads();                                      // the values and the mixed weights are there
     const bf16* tV = buf1 + kvh * TA_KEYS * VS;
-    const float* pw = sP + h * 16 * PS;
+    const float* pw = sP + h * HS;
 #pragma unroll
     for (int kk = 0; kk < 2; ++kk) {
       uint32_t t[3][4];
@@ -459,8 +519,15 @@ __global__ void __launch_bounds__(256) talking_slice_kernel(TalkArgs a, TalkSlic
   float* sS = (float*)(ring + stages * stage_elems);
   float* corr = sS + 16 * SS;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g8 = lane >> 2, tg = lane & 3, mat = lane >> 3, r8 = lane & 7;
-  // what a product may read beyond the rows and columns that exist must be finite
-  for (int i = tid; i < (int)((16 * L.QS + stages * stage_elems) / 8); i += 256) ((uint4*)ta_smem)[i] = make_uint4(0u, 0u, 0u, 0u);
+  // what a product may read beyond the rows and columns that exist must be finite: the queries' other rows and the rows' padding
+  for (int i = tid; i < 16 * L.QS / 8; i += 256) ((uint4*)sQ)[i] = make_uint4(0u, 0u, 0u, 0u);
+  const int kp = (L.KR - G * n) / 8, vp_ = (L.VR - G * dv) / 8;
+  for (int i = tid; i < stages * KB * (kp + vp_); i += 256) {
+    const int row = i / (kp + vp_), c = i % (kp + vp_);
+    bf16* base = ring + (row / KB) * stage_elems;
+    bf16* dst = c < kp ? base + (row % KB) * L.KR + G * n + c * 8 : base + KB * L.KR + (row % KB) * L.VR + G * dv + (c - kp) * 8;
+    *(uint4*)dst = make_uint4(0u, 0u, 0u, 0u);
+  }
   for (int i = tid; i < 16 * SS + 16; i += 256) sS[i] = 0.f;
   __syncthreads();
   pdl_wait();
@@ -482,13 +549,12 @@ __global__ void __launch_bounds__(256) talking_slice_kernel(TalkArgs a, TalkSlic
     const int jr = j0 + (lane & (KB - 1));
     unsigned long long row_at = 0;
     if (jr < k_hi) row_at = ((unsigned long long)bt[jr / page] * page + (unsigned long long)(jr % page)) * width;
-    for (int idx = tid; idx - lane < KB * per; idx += 256) {      // the same number of rounds for every lane of a warp
-      const int r = min(idx / per, KB - 1), c = idx - r * per;
-      const unsigned long long at = __shfl_sync(0xffffffffu, row_at, r);
-      if (idx < KB * per) {
-        const bool valid = j0 + r < k_hi;
-        ta_cp16(c < kc ? dK + r * L.KR + c * 8 : dV + r * L.VR + (c - kc) * 8, valid ? a.cache + at + (size_t)c * 8 : a.cache, valid);
-      }
+    for (int r = warp; r < KB; r += 8) {
+      const bf16* row = a.cache + __shfl_sync(0xffffffffu, row_at, r);
+      const bool valid = j0 + r < k_hi;
+      if (!valid) row = a.cache;
+      for (int c = lane; c < per; c += 32)
+        ta_cp16(c < kc ? dK + r * L.KR + c * 8 : dV + r * L.VR + (c - kc) * 8, row + (valid ? c * 8 : 0), valid);
     }
     ta_commit();
   };
@@ -535,7 +601,7 @@ __global__ void __launch_bounds__(256) talking_slice_kernel(TalkArgs a, TalkSlic
       if (row < H) {
         const float v = lane < KB ? sS[row * SS + lane] : -INFINITY;
         const float mn = fmaxf(m_[half], warp_max(v));    // finite: a block holds a key
-        const float p = exp2f(v - mn), cf = exp2f(m_[half] - mn);
+        const float p = ta_exp2(v - mn), cf = ta_exp2(m_[half] - mn);
         l_[half] = l_[half] * cf + warp_sum(p);
         m_[half] = mn;
         if (lane < KB) sS[row * SS + lane] = p;
@@ -653,14 +719,19 @@ extern "C" int qv_talking_attention_mma(void* out, int ld_out, const void* q, in
   a.capped = cap > 0.f;
   a.pre = a.capped ? 2.0f * TA_LOG2E * scale / cap : TA_LOG2E * scale;
   a.post = a.capped ? cap * TA_LOG2E : 1.0f;
-  a.sink = sink; a.partial = partial; a.slices = slices < 1 ? 1 : slices; a.slice_keys = slice_keys;
+  a.sink = sink; a.talk = talk; a.talk_terms = 1; a.partial = partial;
+  for (int i = 0; i < H * H; ++i) {
+    uint32_t bits;
+    memcpy(&bits, talk_host + i, 4);
+    if (bits & 0xffffu) a.talk_terms = 3;
+  } a.slices = slices < 1 ? 1 : slices; a.slice_keys = slice_keys;
   cudaStream_t st = (cudaStream_t)stream;
   int rc = QV_ERR_UNSUPPORTED;
   if (max_q_len == 1) {
     if (partial == nullptr || slice_keys <= 0 || slice_keys % TA_KEYS || G * dv > 2048) return QV_ERR_UNSUPPORTED;
     const TalkSliceLayout L = ta_slice_layout(G, n, dv);
-    int kb = 32, stages = 2;
-    if (ta_slice_smem(L, 32, 2) > LIMIT) kb = 16;
+    // blocks of 16 keys where two or three CTAs then share an SM (their loads overlap one another's products), else of 32
+    int kb = ta_slice_smem(L, 32, 2) > 56 * 1024 ? 16 : 32, stages = 2;
     if (ta_slice_smem(L, kb, 2) > LIMIT) stages = 1;
     const size_t smem = ta_slice_smem(L, kb, stages);
     if (smem > LIMIT) return QV_ERR_UNSUPPORTED;
@@ -673,9 +744,10 @@ extern "C" int qv_talking_attention_mma(void* out, int ld_out, const void* q, in
     if (kb == 32) {
       if (per_warp <= 2) TA_SLICE(32, 2);
       else if (per_warp <= 8) TA_SLICE(32, 8);
-      else TA_SLICE(32, 32);
+      else return QV_ERR_UNSUPPORTED;                      // (56 KB do not hold so many value columns)
     } else {
       if (per_warp <= 8) TA_SLICE(16, 8);
+      else if (per_warp <= 16) TA_SLICE(16, 16);
       else TA_SLICE(16, 32);
     }
 #undef TA_SLICE
@@ -690,9 +762,10 @@ extern "C" int qv_talking_attention_mma(void* out, int ld_out, const void* q, in
   const size_t stat_off = smem - (size_t)2 * H * 16 * sizeof(float);
 #define TA_TILE(NP_, DP_, HP_)                                                                                                       \
   do {                                                                                                                               \
-    TalkMatrix<HP_> mix;                                                                                                             \
-    for (int h = 0; h < HP_; ++h)                                                                                                    \
-      for (int g = 0; g < HP_; ++g) mix.t[h * HP_ + g] = h < H && g < H ? talk_host[h * H + g] : 0.f;                                \
+    TalkMatrix<(HP_ < 16 ? HP_ : 1)> mix;                                                                                                             \
+    if (HP_ < 16)                                                                                                                    \
+      for (int h = 0; h < HP_; ++h)                                                                                                  \
+        for (int g = 0; g < HP_; ++g) mix.t[HP_ < 16 ? h * HP_ + g : 0] = h < H && g < H ? talk_host[h * H + g] : 0.f;                              \
     cudaFuncSetAttribute(talking_tile_kernel<NP_, DP_, HP_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                \
     rc = qv_launch_cluster(talking_tile_kernel<NP_, DP_, HP_>, dim3((max_q_len + 15) / 16 * cs, 1, S), dim3(32 * H), smem, st,       \
                            dim3(cs, 1, 1), a, mix, cs, stat_off);                                                                    \

@@ -698,7 +698,7 @@ def talking_attention_case(seg_lens, ctx_len, peaks, page=16) -> dict:
     q = torch.randn(T, H * n, device="cuda", dtype=torch.bfloat16)
     out = torch.empty(T, H * dv, device="cuda", dtype=torch.bfloat16)
     sink = torch.randn(H, device="cuda")
-    talk = torch.eye(H) + torch.randn(H, H) * 0.2
+    talk = (torch.eye(H) + torch.randn(H, H) * 0.2).to(torch.bfloat16).float()
     talk_dev = talk.cuda()
     us = kb.timed_chain(lambda i: ops.talking_attention(out, q, caches[i % copies], ctx, table, H, G, n, dv, page, a["scale"], a["softcap"], sink,
                                                         talk_dev, talk), launches=8)

@@ -449,7 +449,8 @@ def test_slices_and_shares_follow_from_the_steps_shape():
     assert ops.talking_attention_slices(1, 4, 64, 100) == (4, 32)
     slices, keys = ops.talking_attention_slices(64, 16, 512, 1 << 17)
     assert slices * keys >= 1 << 17 and 64 * slices * 16 * 514 * 4 <= 128 << 20
-    assert ops.talking_attention_cluster(1) == 8 and ops.talking_attention_cluster(1000) == 1
+    assert ops.talking_attention_cluster([2], [40]) == 8 and ops.talking_attention_cluster([16] * 1000, [0] * 1000) == 1
+    assert ops.talking_attention_cluster([2048], [0]) in (2, 4) and ops.talking_attention_cluster([512], [1536]) in (4, 8)
 
 
 # ---------------------------------------------------------------------------------------------- delta rule
