@@ -331,7 +331,7 @@ extern "C" int qv_head_delta_scan(float* out, int ld_out, const float* qn, const
   const int row = 2 * HD_PAD * lpc + HD_COEF + cta_cols;
   int chunk = max_q_len <= 1 ? 1 : (max_q_len > 32 ? 32 : (max_q_len + 3) / 4 * 4);
   while (chunk > HD_BLOCK && (size_t)2 * chunk * row * sizeof(float) > 96 * 1024) chunk -= HD_BLOCK;
-  if (block > 1 && chunk < HD_BLOCK) chunk = HD_BLOCK;
+  if (block > 1 && max_q_len > 1 && chunk < HD_BLOCK) chunk = HD_BLOCK;
   const size_t smem = (size_t)2 * chunk * row * sizeof(float);
   const int vec4 = dk % 4 == 0 && (((uintptr_t)qn | (uintptr_t)kn) & 15) == 0;
   if (((uintptr_t)coef) & 15) return QV_ERR_UNSUPPORTED;
@@ -341,10 +341,10 @@ extern "C" int qv_head_delta_scan(float* out, int ld_out, const float* qn, const
     if (max_q_len >= 16) return hd_launch_after(head_delta_scan_kernel<LPC_, B_>, grid, blk, smem, st, a, chunk, vec4);      \
     return qv_launch(head_delta_scan_kernel<LPC_, B_>, grid, blk, smem, st, a, chunk, vec4);                                 \
   } while (0)
-#define HD_BLOCKS(LPC_)                          \
-  do {                                           \
-    if (block == 1) HD_LAUNCH(LPC_, 1);          \
-    HD_LAUNCH(LPC_, HD_BLOCK);                   \
+#define HD_BLOCKS(LPC_)                                   \
+  do {                                                    \
+    if (block == 1 || max_q_len <= 1) HD_LAUNCH(LPC_, 1); \
+    HD_LAUNCH(LPC_, HD_BLOCK);                            \
   } while (0)
   if (lpc == 1) HD_BLOCKS(1);
   if (lpc == 2) HD_BLOCKS(2);

@@ -960,7 +960,7 @@ def talking_attention_slices(tokens: int, H: int, values: int, max_ctx: int):
     """(slices, keys a slice) for single query tokens (a CTA serves a token and a slice; a slice leaves H x `values` partial
     sums): few tokens still fill the SMs, the slices cover the longest context the step may hold, and their partial sums stay
     within some hundred megabytes."""
-    keys = 32 if tokens <= 2 else 64 if tokens <= 16 else 128 if tokens <= 64 else 256
+    keys = 64 if tokens <= 16 else 128 if tokens <= 64 else 256
     while tokens * -(-max_ctx // keys) * H * (values + 2) * 4 > 128 << 20 and keys < max_ctx:
         keys *= 2
     return max(1, -(-max_ctx // keys)), keys

@@ -15,8 +15,9 @@
 //                                with the values as three bfloat16 terms that together hold their 24 bits):
 //   portions       a cluster of CTAs owns 16 consecutive tokens and all heads (a warp a head); its CTAs share out the blocks of 32
 //                  keys.  Pass 1: every head's maximum and sum, joined over the cluster through distributed shared memory.  Pass 2:
-//                  the normalised weights of a block go to shared memory, a thread mixes all heads of one (query, key), and a warp
-//                  multiplies its head's mixed weights with the values; at the end the cluster's partial outputs are added in rank order.
+//                  the normalised weights of a block go to shared memory and are mixed in place (up to eight heads: a thread mixes all
+//                  heads of one (query, key); more: products of the matrix with the weights of eight pairs on the tensor cores, the
+//                  weights as three bfloat16 terms), and a warp multiplies its head's mixed weights with the values; at the end the cluster's partial outputs are added in rank order.
 //   single tokens  a CTA owns one token and a slice of its keys, with the heads as the tile's rows.  Since mixing is linear,
 //                      out_h = sum_g talk[h, g] / L_g * (sum_j exp(s_g(j)) v_j,kv(h)),
 //                  a slice multiplies every head's unnormalised weights with the values of ALL key/value heads (read once), and
@@ -561,7 +562,8 @@ __global__ void __launch_bounds__(256) talking_slice_kernel(TalkArgs a, TalkSlic
   float o[CT][4];
 #pragma unroll
   for (int i = 0; i < CT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  float m_[2] = {-INFINITY, -INFINITY}, l_[2] = {0.f, 0.f};        // rows warp and warp + 8
+  constexpr int RW = KB == 16 ? 1 : 2;
+  float m_[2] = {-INFINITY, -INFINITY}, l_[2] = {0.f, 0.f};
   const int nt_all = vc, nt0 = warp * CT;
   const int nkb = (k_hi - k_lo + KB - 1) / KB, n16 = (n + 15) / 16;
   load(0, k_lo);
@@ -595,17 +597,21 @@ __global__ void __launch_bounds__(256) talking_slice_kernel(TalkArgs a, TalkSlic
         }
     }
     __syncthreads();
+    // a lane keeps its share of a row's sum; blocks of 16 keys: a row each half of the warp, else the warp's two rows one by one
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int row = warp + half * 8;
+    for (int x = 0; x < RW; ++x) {
+      const int row = KB == 16 ? 2 * warp + (lane >> 4) : warp + x * 8, key = lane & (KB - 1);
+      const float v = row < H ? sS[row * SS + key] : 0.f;
+      float mn = v;
+#pragma unroll
+      for (int o2 = KB / 2; o2 > 0; o2 >>= 1) mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, o2));
+      mn = fmaxf(mn, m_[x]);                              // finite: a block holds a key
+      const float p = ta_exp2(v - mn), cf = ta_exp2(m_[x] - mn);
+      l_[x] = l_[x] * cf + p;
+      m_[x] = mn;
       if (row < H) {
-        const float v = lane < KB ? sS[row * SS + lane] : -INFINITY;
-        const float mn = fmaxf(m_[half], warp_max(v));    // finite: a block holds a key
-        const float p = ta_exp2(v - mn), cf = ta_exp2(m_[half] - mn);
-        l_[half] = l_[half] * cf + warp_sum(p);
-        m_[half] = mn;
-        if (lane < KB) sS[row * SS + lane] = p;
-        if (lane == 0) corr[row] = cf;
+        sS[row * SS + key] = p;
+        if (key == 0) corr[row] = cf;
       }
     }
     __syncthreads();
@@ -641,9 +647,11 @@ __global__ void __launch_bounds__(256) talking_slice_kernel(TalkArgs a, TalkSlic
   const int stride = 2 + G * dv;
   float* part = a.partial + ((size_t)s * a.slices + blockIdx.x) * H * stride;
 #pragma unroll
-  for (int half = 0; half < 2; ++half) {
-    const int row = warp + half * 8;
-    if (row < H && lane == 0) { part[(size_t)row * stride] = m_[half]; part[(size_t)row * stride + 1] = l_[half]; }
+  for (int x = 0; x < RW; ++x) {
+    const int row = KB == 16 ? 2 * warp + (lane >> 4) : warp + x * 8;
+#pragma unroll
+    for (int o2 = KB / 2; o2 > 0; o2 >>= 1) l_[x] += __shfl_xor_sync(0xffffffffu, l_[x], o2);
+    if (row < H && (lane & (KB - 1)) == 0) { part[(size_t)row * stride] = m_[x]; part[(size_t)row * stride + 1] = l_[x]; }
   }
 #pragma unroll
   for (int i = 0; i < CT; ++i) {
@@ -655,8 +663,8 @@ __global__ void __launch_bounds__(256) talking_slice_kernel(TalkArgs a, TalkSlic
 }
 
 // joins a token's slices (ascending), divides by the sums (with the sink's share) and mixes.  A CTA takes 32 of the G * dv value
-// columns' worth of one key/value head; a warp joins the slices of every eighth head, then the head's outputs are mixed.
-__global__ void __launch_bounds__(256) talking_merge_kernel(bf16* __restrict__ out, int ld_out, const float* __restrict__ partial,
+// columns' worth of one key/value head; a warp joins the slices of a head, then the head's outputs are mixed.
+__global__ void __launch_bounds__(512) talking_merge_kernel(bf16* __restrict__ out, int ld_out, const float* __restrict__ partial,
                                                            const int* __restrict__ seg_q_start, const int* __restrict__ seg_pos0, int H,
                                                            int G, int dv, int all_slices, int slice_keys, const float* __restrict__ sink,
                                                            const float* __restrict__ talk) {
@@ -669,7 +677,7 @@ __global__ void __launch_bounds__(256) talking_merge_kernel(bf16* __restrict__ o
   const size_t step = (size_t)H * stride;
   const float* p = partial + (size_t)s * all_slices * step;
   const int slices = min(all_slices, seg_pos0[s] / slice_keys + 1);       // the slices that hold keys of this token
-  for (int g = warp; g < H; g += 8) {
+  for (int g = warp; g < H; g += 16) {
     const float* pg = p + (size_t)g * stride;
     const float snk = sink[g] * TA_LOG2E;
     float M = snk, L = 0.f, acc = 0.f;
@@ -680,7 +688,7 @@ __global__ void __launch_bounds__(256) talking_merge_kernel(bf16* __restrict__ o
       const float wi = in ? exp2f(pg[(size_t)(base + lane) * step] - M) : 0.f;
       L += in ? pg[(size_t)(base + lane) * step + 1] * wi : 0.f;
       const int cnt = min(32, slices - base);
-#pragma unroll 8
+#pragma unroll 16
       for (int j = 0; j < cnt; ++j) {
         const float wj = __shfl_sync(0xffffffffu, wi, j);
         if (col < dv) acc = fmaf(pg[(size_t)(base + j) * step + 2 + (size_t)c * dv + col], wj, acc);
@@ -692,7 +700,7 @@ __global__ void __launch_bounds__(256) talking_merge_kernel(bf16* __restrict__ o
   __syncthreads();
   bf16* orow = out + (size_t)seg_q_start[s] * ld_out;
   if (col < dv)
-    for (int hh = warp; hh < gs; hh += 8) {
+    for (int hh = warp; hh < gs; hh += 16) {
       const int h = c * gs + hh;
       float w = 0.f;
       for (int g = 0; g < H; ++g) w = fmaf(talk[(size_t)h * H + g], R[g][lane], w);
@@ -752,7 +760,7 @@ extern "C" int qv_talking_attention_mma(void* out, int ld_out, const void* q, in
     }
 #undef TA_SLICE
     if (rc) return rc;
-    return qv_launch(talking_merge_kernel, dim3(S, G * ((dv + 31) / 32)), dim3(256), 0, st, (bf16*)out, ld_out, (const float*)partial,
+    return qv_launch(talking_merge_kernel, dim3(S, G * ((dv + 31) / 32)), dim3(512), 0, st, (bf16*)out, ld_out, (const float*)partial,
                      seg_q_start, seg_pos0, H, G, dv, a.slices, slice_keys, sink, talk);
   }
   if (cs != 1 && cs != 2 && cs != 4 && cs != 8) return QV_ERR_UNSUPPORTED;

@@ -446,7 +446,7 @@ def test_slices_of_single_tokens(H, G, n, dv, keys):
 
 def test_slices_and_shares_follow_from_the_steps_shape():
     assert ops.talking_attention_slices(8, 16, 512, 1024) == (16, 64)
-    assert ops.talking_attention_slices(1, 4, 64, 100) == (4, 32)
+    assert ops.talking_attention_slices(1, 4, 64, 100) == (2, 64)
     slices, keys = ops.talking_attention_slices(64, 16, 512, 1 << 17)
     assert slices * keys >= 1 << 17 and 64 * slices * 16 * 514 * 4 <= 128 << 20
     assert ops.talking_attention_cluster([2], [40]) == 8 and ops.talking_attention_cluster([16] * 1000, [0] * 1000) == 1
