@@ -2,8 +2,8 @@
 //   a_m = softmax_j((q_m . k_m,j) * scale) V      for the two maps m = 1, 2 (causal, optionally the last `window` keys),
 //   o = a_1 - lam * a_2;   out = o / sqrt(mean(o^2) + eps) * post            (mean over the head's value entries).
 //
-// qv_diff_prepare            per token (a CTA): bias added to the projection's sums, every map of q and k divided by its
-//                            root mean square and weighted, the first `rot` entries of each map rotated (pairs i, i + rot/2,
+// qv_diff_prepare            per token (a CTA): bias (if any) added to the projection's sums, every map of q and k divided by its
+//                            root mean square and weighted (where there are weights qw, kw), the first `rot` entries of each map rotated (pairs i, i + rot/2,
 //                            cos/sin from a table row of the token's position); q goes to a dense buffer, k and v (with
 //                            its bias) to the token's cache row [k: G x 2n | v: G x dv].  All arithmetic float32.
 // qv_diff_attention_generic  one warp per (token, head), float32 arithmetic whatever the storage type, any sizes; keys in
@@ -58,20 +58,23 @@ __global__ void __launch_bounds__(256) diff_prepare_kernel(T* __restrict__ q_out
       if (!is_q && !crow) continue;
       const int col0 = unit * n;                             // the k maps follow the q maps in the projection's columns
       const float* src = prep_row + col0;
-      float ss = 0.f;
-      for (int i = lane; i < n; i += 32) ss = fmaf(src[i], src[i], ss);
-      ss = warp_sum(ss);
-      const float inv = 1.0f / sqrtf(ss / (float)n + eps);
       const float* w = is_q ? qw : kw;
+      float inv = 1.0f;
+      if (w) {
+        float ss = 0.f;
+        for (int i = lane; i < n; i += 32) ss = fmaf(src[i], src[i], ss);
+        ss = warp_sum(ss);
+        inv = 1.0f / sqrtf(ss / (float)n + eps);
+      }
       T* dst = is_q ? q_out + (size_t)t * ld_q + col0 : crow + (size_t)(unit - nq) * n;
       for (int i = lane; i < half; i += 32) {
-        const float u = src[i] * inv * w[i];
-        const float v = src[i + half] * inv * w[i + half];
+        const float u = src[i] * inv * (w ? w[i] : 1.0f);
+        const float v = src[i + half] * inv * (w ? w[i + half] : 1.0f);
         const float2 c = cs[i];
         dst[i] = from_f<T>(u * c.x - v * c.y);
         dst[i + half] = from_f<T>(v * c.x + u * c.y);
       }
-      for (int i = rot + lane; i < n; i += 32) dst[i] = from_f<T>(src[i] * inv * w[i]);
+      for (int i = rot + lane; i < n; i += 32) dst[i] = from_f<T>(src[i] * inv * (w ? w[i] : 1.0f));
     } else if (crow) {
       const int vh = unit - nq - nk;
       const float* src = prep_row + (nq + nk) * n + vh * dv;

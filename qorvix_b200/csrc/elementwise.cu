@@ -523,29 +523,43 @@ extern "C" int qv_add_vector(float* x, const float* v, int T, int d, void* strea
 }
 
 // ---------------------------------------------------------------- ungated activations
-// out = act(x) elementwise in place or not; kind 0: the square of relu, 1: the tanh form of GELU.
-template <typename T>
-__global__ void activation_kernel(T* __restrict__ out, const T* __restrict__ x, size_t n, int kind) {
+// out = act(x + bias) elementwise in place or not, bias one number per column of rows of `cols` (or null); kind 0: the square of
+// relu, 1: the tanh form of GELU.  VEC elements at a time (VEC 4: n and cols multiples of 4, pointers on the vectors' boundaries).
+__device__ __forceinline__ float activation_of(float z, int kind) {
+  if (kind == 1) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  const float v = fmaxf(z, 0.f);
+  return v * v;
+}
+
+template <typename T, int VEC>
+__global__ void activation_kernel(T* out, const T* x, const float* __restrict__ bias, size_t n, int cols, int kind) {
   pdl_wait();
   pdl_launch_dependents();
-  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
-    const float z = to_f(x[i]);
-    float r;
-    if (kind == 1) {
-      r = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  for (size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * VEC; i < n; i += (size_t)gridDim.x * blockDim.x * VEC) {
+    const int c = bias ? (int)(i % (unsigned)cols) : 0;
+    if constexpr (VEC == 4) {
+      float4 z = Vec4<T>::load(x + i);
+      if (bias) {
+        const float4 b = *(const float4*)(bias + c);
+        z.x += b.x; z.y += b.y; z.z += b.z; z.w += b.w;
+      }
+      store4(out + i, make_float4(activation_of(z.x, kind), activation_of(z.y, kind), activation_of(z.z, kind), activation_of(z.w, kind)));
     } else {
-      const float v = fmaxf(z, 0.f);
-      r = v * v;
+      out[i] = from_f<T>(activation_of(to_f(x[i]) + (bias ? bias[c] : 0.f), kind));
     }
-    out[i] = from_f<T>(r);
   }
 }
 
-extern "C" int qv_activation(void* out, const void* x, long long n, int kind, int dt, void* stream) {
+extern "C" int qv_activation(void* out, const void* x, const float* bias, long long n, int cols, int kind, int dt, void* stream) {
   if (n <= 0) return 0;
-  if (kind != 0 && kind != 1) return QV_ERR_UNSUPPORTED;
-  const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
-  QV_DISPATCH_DT(dt, TT, return qv_launch(activation_kernel<TT>, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (TT*)out, (const TT*)x, (size_t)n, kind));
+  if ((kind != 0 && kind != 1) || cols <= 0) return QV_ERR_UNSUPPORTED;
+  const bool vec = n % 4 == 0 && cols % 4 == 0 && (((uintptr_t)out | (uintptr_t)x | (uintptr_t)bias) & 15) == 0;
+  const long long work = vec ? n / 4 : n;
+  const int blocks = (int)((work + 255) / 256 < 148 * 16 ? (work + 255) / 256 : 148 * 16);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (vec)
+    QV_DISPATCH_DT(dt, TT, return qv_launch(activation_kernel<TT, 4>, dim3(blocks), dim3(256), 0, st, (TT*)out, (const TT*)x, bias, (size_t)n, cols, kind));
+  QV_DISPATCH_DT(dt, TT, return qv_launch(activation_kernel<TT, 1>, dim3(blocks), dim3(256), 0, st, (TT*)out, (const TT*)x, bias, (size_t)n, cols, kind));
   return QV_ERR_UNSUPPORTED;
 }
 
@@ -845,5 +859,187 @@ extern "C" int qv_rmsnorm_rows(void* out, int ld_out, const void* in, int ld_in,
   if (in_dt == QV_DT_F32 && out_dt == QV_DT_BF16) LAUNCH_ROWS(float, bf16);
   if (in_dt == QV_DT_BF16 && out_dt == QV_DT_F32) LAUNCH_ROWS(bf16, float);
 #undef LAUNCH_ROWS
+  return QV_ERR_UNSUPPORTED;
+}
+
+// ---------------------------------------------------------------- several residual streams (hyper-connections)
+// The residual is S streams, streams[t][s][:] float32.  A sublayer's input is u = sum_s in[s] x_s; its output y goes back as
+// x_t <- sum_s mix[s][t] x_s + out[t] (y + y_bias), all streams at once from the old ones.  One pass does the write that is still
+// pending and the read of the sublayer that comes next:
+//   old x_s from `streams`, or, with x0, the one row x0[t] for all of them (the embedding's output, ahead of the first sublayer);
+//   with write_coef ([S][S] mix, then [S] out): the write above, y in the compute type or float32 (row stride ld_y);
+//   with `store`: the streams as they now are go to `streams`;
+//   out = u, or with a weight w the norm of it: u / sqrt(mean(u^2) + eps) * w;   read_coef: [S] in.
+// Row r of out belongs to token row_idx[r] (or r).  One block per row; the sums' order depends on d and S alone.
+// NS > 0: the number of streams; NS 0: any up to 16.  VEC: four entries at a time, u kept in registers (d a multiple of 4, at
+// most 4 * 4 * 256 entries, pointers and rows on 16 bytes); else u lies in shared memory.
+#define STREAMS_MAX 16
+template <typename TY, typename TO, int NS, bool VEC>
+__global__ void __launch_bounds__(256) stream_pass_kernel(TO* __restrict__ out, float* __restrict__ streams, const float* __restrict__ x0,
+                                                          const TY* __restrict__ y, int ld_y, const float* __restrict__ y_bias,
+                                                          const float* __restrict__ write_coef, const float* __restrict__ read_coef,
+                                                          const float* __restrict__ w, float eps, const int* __restrict__ row_idx,
+                                                          int n_streams, int d, int store) {
+  extern __shared__ float stream_u[];                        // !VEC: d entries of u
+  __shared__ float red[33];
+  __shared__ float cf[STREAMS_MAX * STREAMS_MAX + 2 * STREAMS_MAX];
+  const int S = NS > 0 ? NS : n_streams;
+  float* c_out = cf + S * S;
+  float* c_in = c_out + S;
+  for (int i = threadIdx.x; i < S * S + S; i += 256) cf[i] = write_coef ? write_coef[i] : 0.f;      // weights: no kernel writes them
+  for (int i = threadIdx.x; i < S; i += 256) c_in[i] = read_coef[i];
+  __syncthreads();
+  pdl_wait();
+  pdl_launch_dependents();
+  const int r = blockIdx.x;
+  const int t = row_idx ? row_idx[r] : r;
+  float* xr = streams + (size_t)t * S * d;
+  const float* x0r = x0 ? x0 + (size_t)t * d : nullptr;
+  const TY* yr = write_coef ? y + (size_t)t * ld_y : nullptr;
+  TO* o = out + (size_t)r * d;
+  float ss = 0.f;
+  if constexpr (VEC && NS > 0) {
+    constexpr int MAXV = 4;
+    float4 u[MAXV];
+    const int nvec = d >> 2;
+#pragma unroll
+    for (int k = 0; k < MAXV; ++k) {
+      const int i = threadIdx.x + k * 256;
+      u[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < nvec) {
+        float4 x[NS];
+#pragma unroll
+        for (int s = 0; s < NS; ++s) x[s] = *(const float4*)((x0r ? x0r : xr + (size_t)s * d) + 4 * i);
+        if (yr) {
+          float4 v = Vec4<TY>::load(yr + 4 * i);
+          if (y_bias) {
+            const float4 b = *(const float4*)(y_bias + 4 * i);
+            v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+          }
+          float4 nx[NS];
+#pragma unroll
+          for (int to = 0; to < NS; ++to) {
+            float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int s = 0; s < NS; ++s) {
+              const float m = cf[s * NS + to];
+              a.x = fmaf(m, x[s].x, a.x); a.y = fmaf(m, x[s].y, a.y); a.z = fmaf(m, x[s].z, a.z); a.w = fmaf(m, x[s].w, a.w);
+            }
+            const float g = c_out[to];
+            a.x = fmaf(g, v.x, a.x); a.y = fmaf(g, v.y, a.y); a.z = fmaf(g, v.z, a.z); a.w = fmaf(g, v.w, a.w);
+            nx[to] = a;
+          }
+#pragma unroll
+          for (int s = 0; s < NS; ++s) x[s] = nx[s];
+        }
+#pragma unroll
+        for (int s = 0; s < NS; ++s) {
+          if (store) *(float4*)(xr + (size_t)s * d + 4 * i) = x[s];
+          const float g = c_in[s];
+          u[k].x = fmaf(g, x[s].x, u[k].x); u[k].y = fmaf(g, x[s].y, u[k].y); u[k].z = fmaf(g, x[s].z, u[k].z); u[k].w = fmaf(g, x[s].w, u[k].w);
+        }
+        if (!w) store4(o + 4 * i, u[k]);
+        ss += u[k].x * u[k].x + u[k].y * u[k].y + u[k].z * u[k].z + u[k].w * u[k].w;
+      }
+    }
+    if (!w) return;
+    const float scale = 1.0f / sqrtf(block_sum(ss, red) / (float)d + eps);
+#pragma unroll
+    for (int k = 0; k < MAXV; ++k) {
+      const int i = threadIdx.x + k * 256;
+      if (i < nvec) {
+        const float4 wv = *(const float4*)(w + 4 * i);
+        store4(o + 4 * i, make_float4(u[k].x * scale * wv.x, u[k].y * scale * wv.y, u[k].z * scale * wv.z, u[k].w * scale * wv.w));
+      }
+    }
+  } else {
+    for (int i = threadIdx.x; i < d; i += 256) {
+      float x[STREAMS_MAX];
+#pragma unroll
+      for (int s = 0; s < STREAMS_MAX; ++s) x[s] = s < S ? (x0r ? x0r[i] : xr[(size_t)s * d + i]) : 0.f;
+      const float v = yr ? to_f(yr[i]) + (y_bias ? y_bias[i] : 0.f) : 0.f;
+      float u = 0.f;
+      for (int to = 0; to < S; ++to) {
+        float a = 0.f;
+        if (yr) {
+#pragma unroll
+          for (int s = 0; s < STREAMS_MAX; ++s)
+            if (s < S) a = fmaf(cf[s * S + to], x[s], a);
+          a = fmaf(c_out[to], v, a);
+        } else {
+          a = x0r ? x0r[i] : xr[(size_t)to * d + i];
+        }
+        if (store) xr[(size_t)to * d + i] = a;
+        u = fmaf(c_in[to], a, u);
+      }
+      if (w) stream_u[i] = u;
+      else o[i] = from_f<TO>(u);
+      ss += u * u;
+    }
+    if (!w) return;
+    const float scale = 1.0f / sqrtf(block_sum(ss, red) / (float)d + eps);
+    for (int i = threadIdx.x; i < d; i += 256) o[i] = from_f<TO>(stream_u[i] * scale * w[i]);
+  }
+}
+
+extern "C" int qv_stream_pass(void* out, float* streams, const float* x0, const void* y, int ld_y, const float* y_bias,
+                              const float* write_coef, const float* read_coef, const float* w, float eps, const int* row_idx, int rows,
+                              int S, int d, int store, int y_dt, int out_dt, void* stream) {
+  if (rows <= 0 || d <= 0) return 0;
+  if (S <= 0 || S > STREAMS_MAX || (row_idx && store) || (write_coef && !y)) return QV_ERR_UNSUPPORTED;
+  cudaStream_t st = (cudaStream_t)stream;
+  const uintptr_t all = (uintptr_t)out | (uintptr_t)streams | (uintptr_t)x0 | (uintptr_t)y | (uintptr_t)y_bias | (uintptr_t)w;
+  const bool vec = S <= 4 && d % 4 == 0 && d <= 4 * 4 * 256 && ld_y % 4 == 0 && (all & 15) == 0;
+  const size_t smem = vec || !w ? 0 : (size_t)d * sizeof(float);
+  if (smem > 200 * 1024) return QV_ERR_TOO_LARGE;
+#define STREAM_GO(TY, TO, N_, V_)                                                                                                  \
+  do {                                                                                                                             \
+    if (smem > 44 * 1024) cudaFuncSetAttribute(stream_pass_kernel<TY, TO, N_, V_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    return qv_launch(stream_pass_kernel<TY, TO, N_, V_>, dim3(rows), dim3(256), smem, st, (TO*)out, streams, x0, (const TY*)y, ld_y, \
+                     y_bias, write_coef, read_coef, w, eps, row_idx, S, d, store);                                                 \
+  } while (0)
+#define STREAM_BY_COUNT(TY, TO)             \
+  do {                                      \
+    if (!vec) STREAM_GO(TY, TO, 0, false);  \
+    if (S == 1) STREAM_GO(TY, TO, 1, true); \
+    if (S == 2) STREAM_GO(TY, TO, 2, true); \
+    if (S == 3) STREAM_GO(TY, TO, 3, true); \
+    STREAM_GO(TY, TO, 4, true);             \
+  } while (0)
+  if (y_dt == QV_DT_F32 && out_dt == QV_DT_F32) STREAM_BY_COUNT(float, float);
+  if (y_dt == QV_DT_BF16 && out_dt == QV_DT_BF16) STREAM_BY_COUNT(bf16, bf16);
+  if (y_dt == QV_DT_F32 && out_dt == QV_DT_BF16) STREAM_BY_COUNT(float, bf16);
+  if (y_dt == QV_DT_BF16 && out_dt == QV_DT_F32) STREAM_BY_COUNT(bf16, float);
+#undef STREAM_BY_COUNT
+#undef STREAM_GO
+  return QV_ERR_UNSUPPORTED;
+}
+
+// ---------------------------------------------------------------- rows into the paged cache
+// cache row of token t (its page and place from the block table) = src[t, :width], the types being equal.  One block per token.
+template <typename T>
+__global__ void __launch_bounds__(128) cache_rows_kernel(T* __restrict__ cache, const T* __restrict__ src, int ld, const int* __restrict__ tok_pos,
+                                                         const int* __restrict__ tok_seg, const int* __restrict__ block_table,
+                                                         int max_blocks, int width, int page) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x, pos = tok_pos[t];
+  const int pg = block_table[(size_t)tok_seg[t] * max_blocks + pos / page];
+  T* dst = cache + ((size_t)pg * page + (size_t)(pos % page)) * width;
+  const T* s = src + (size_t)t * ld;
+  constexpr int PER = 16 / (int)sizeof(T);
+  if (width % PER == 0 && (((uintptr_t)dst | (uintptr_t)s) & 15) == 0) {
+    for (int i = threadIdx.x; i < width / PER; i += 128) ((uint4*)dst)[i] = ((const uint4*)s)[i];
+  } else {
+    for (int i = threadIdx.x; i < width; i += 128) dst[i] = s[i];
+  }
+}
+
+extern "C" int qv_cache_rows(void* cache, const void* src, int ld, const int* tok_pos, const int* tok_seg, const int* block_table,
+                             int max_blocks, int T, int width, int page, int dt, void* stream) {
+  if (T <= 0) return 0;
+  if (width <= 0 || page <= 0) return QV_ERR_UNSUPPORTED;
+  QV_DISPATCH_DT(dt, TT, return qv_launch(cache_rows_kernel<TT>, dim3(T), dim3(128), 0, (cudaStream_t)stream, (TT*)cache, (const TT*)src, ld,
+                                          tok_pos, tok_seg, block_table, max_blocks, width, page));
   return QV_ERR_UNSUPPORTED;
 }

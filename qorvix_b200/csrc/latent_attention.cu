@@ -6,7 +6,8 @@
 //   out(t)      = Wuv_h (sum_j p_j c_j)
 // so a query is first carried into the latent space (rank entries), attention then runs as if all heads
 // shared one key/value head whose key row is [c | kr] and whose value row is c, and the head's value
-// matrix is applied to the weighted latent afterwards.  A sigmoid gate multiplies the output.
+// matrix is applied to the weighted latent afterwards.  A sigmoid gate multiplies the output, where there is one; the softmax'
+// denominator takes exp(sink[h]) too, where there are sinks; without a rotated part dr is 0.
 //
 // qv_latent_prepare: per token, RMS norm of the latent part of the down projection, rotation of the shared
 //   key part (neighbouring pairs or split halves), write of both into the token's cache row; rotation of
@@ -93,7 +94,7 @@ __global__ void __launch_bounds__(128) latent_attention_generic_kernel(
     T* __restrict__ out, int ld_out, const T* __restrict__ q, int ld_q, const T* __restrict__ gate, int ld_gate,
     const T* __restrict__ cache, const TW* __restrict__ wuk, const TW* __restrict__ wuv, const int* __restrict__ tok_pos,
     const int* __restrict__ tok_seg, const int* __restrict__ block_table, int max_blocks, int H, int dn, int dr, int dv,
-    int rank, int page, int window, float scale) {
+    int rank, int page, int window, float scale, const float* __restrict__ sink) {
   extern __shared__ float sm_all[];              // 4 warps x (rank + dr + dn) floats
   pdl_wait();
   pdl_launch_dependents();
@@ -123,7 +124,7 @@ __global__ void __launch_bounds__(128) latent_attention_generic_kernel(
   float o[NREG];
 #pragma unroll
   for (int j = 0; j < NREG; ++j) o[j] = 0.f;
-  float m = -INFINITY, l = 0.f;
+  float m = sink ? sink[h] : -INFINITY, l = sink ? 1.f : 0.f;      // a sink: a key of score sink[h] without a value
   for (int kb = (lo >> 5) << 5; kb <= pos; kb += 32) {
     const int tk = kb + lane;
     const bool valid = tk >= lo && tk <= pos;
@@ -183,7 +184,7 @@ extern "C" int qv_latent_attention_generic(void* out, int ld_out, const void* q,
                                            const void* cache, const void* wuk, const void* wuv, const int* tok_pos,
                                            const int* tok_seg, const int* block_table, int max_blocks, int T, int H, int dn,
                                            int dr, int dv, int rank, int page, int window, float scale, int dt, int w_dt,
-                                           void* stream) {
+                                           const float* sink, void* stream) {
   if (T <= 0) return 0;
   if (rank > LAT_MAX_RANK || rank <= 0 || dn < 0 || dr < 0 || dv <= 0) return QV_ERR_UNSUPPORTED;
   const size_t smem = (size_t)4 * (rank + dr + dn) * sizeof(float);
@@ -204,7 +205,7 @@ extern "C" int qv_latent_attention_generic(void* out, int ld_out, const void* q,
       cudaFuncSetAttribute(latent_attention_generic_kernel<TT, TW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     rc = qv_launch(latent_attention_generic_kernel<TT, TW>, grid, dim3(128), smem, st, (TT*)o, ld_out, (const TT*)qq, ld_q, \
                    (const TT*)gg, ld_gate, (const TT*)cache, (const TW*)wuk, (const TW*)wuv, tok_pos + done, tok_seg + done, \
-                   block_table, max_blocks, H, dn, dr, dv, rank, page, window, scale);                                   \
+                   block_table, max_blocks, H, dn, dr, dv, rank, page, window, scale, sink);                             \
   } while (0)
     if (dt == QV_DT_F32 && w_dt == QV_DT_F32) LAT_GENERIC(float, float);
     else if (dt == QV_DT_BF16 && w_dt == QV_DT_BF16) LAT_GENERIC(bf16, bf16);
@@ -224,7 +225,8 @@ extern "C" int qv_latent_attention_generic(void* out, int ld_out, const void* q,
 // sharing the cache rows as keys ([c | kr]) and as values (c): a CTA of eight warps takes 32 consecutive
 // (token, head) rows of one segment and walks its keys in blocks of 64 staged by cp.async in two buffers;
 // Q.K^T and P.V are mma.sync m16n8k16 with float32 accumulators, the softmax is float32 with a running
-// maximum; the keys of a tile may be split over several CTAs, each leaving an unnormalised partial result;
+// maximum, its weights entering P.V as WT bfloat16 terms (1: rounded; 3: terms that together hold a weight's 24 bits);
+// the keys of a tile may be split over several CTAs, each leaving an unnormalised partial result;
 // (3) qv_latent_expand merges the partial results, applies the head's value matrix and the gate.
 #define LT_BM 32
 #define LT_BK 64
@@ -334,7 +336,7 @@ __global__ void __launch_bounds__(128) heads_gemm_kernel(bf16* __restrict__ out,
     }
 }
 
-template <int NTW>
+template <int NTW, int WT>
 __global__ void __launch_bounds__(LT_WARPS * 32) latent_attention_tc_kernel(
     float* __restrict__ part_o, float* __restrict__ part_ml, const bf16* __restrict__ qlat, const bf16* __restrict__ cache,
     const int* __restrict__ seg_q_start, const int* __restrict__ seg_pos0, const int* __restrict__ block_table, int max_blocks,
@@ -344,8 +346,9 @@ __global__ void __launch_bounds__(LT_WARPS * 32) latent_attention_tc_kernel(
   const int kw = RANK + dr, ldk = kw + 8;
   bf16* Qs = (bf16*)lt_smem;                               // [32][ldk]
   bf16* Ks = Qs + (size_t)LT_BM * ldk;                     // [2][64][ldk]
-  bf16* Ps = Ks + (size_t)2 * LT_BK * ldk;                 // [32][72]
-  float* st_max = (float*)(Ps + LT_BM * (LT_BK + 8));      // [8][32]
+  constexpr int PLANE = LT_BM * (LT_BK + 8);               // one term of the weights
+  bf16* Ps = Ks + (size_t)2 * LT_BK * ldk;                 // [WT][32][72]
+  float* st_max = (float*)(Ps + WT * PLANE);               // [8][32]
   float* st_sum = st_max + LT_WARPS * LT_BM;               // [8][32]
   pdl_wait();
   pdl_launch_dependents();
@@ -469,7 +472,16 @@ __global__ void __launch_bounds__(LT_WARPS * 32) latent_attention_tc_kernel(
         corr[mt][hf] = expf(m_run[mt][hf] - m_use);
         m_run[mt][hf] = m_new;
         const float p0 = expf(sc[mt][hf * 2] - m_use), p1 = expf(sc[mt][hf * 2 + 1] - m_use);
-        *(__nv_bfloat162*)(Ps + (size_t)r * (LT_BK + 8) + warp * 8 + 2 * (lane & 3)) = __floats2bfloat162_rn(p0, p1);
+        {
+          float w0 = p0, w1 = p1;
+#pragma unroll
+          for (int term = 0; term < WT; ++term) {            // the weight rounded, then what is left, rounded again, ...
+            const __nv_bfloat162 pr = __floats2bfloat162_rn(w0, w1);
+            *(__nv_bfloat162*)(Ps + term * PLANE + (size_t)r * (LT_BK + 8) + warp * 8 + 2 * (lane & 3)) = pr;
+            w0 -= __low2float(pr);
+            w1 -= __high2float(pr);
+          }
+        }
         float sum = p0 + p1;
         sum += __shfl_xor_sync(0xffffffffu, sum, 1);
         sum += __shfl_xor_sync(0xffffffffu, sum, 2);
@@ -491,15 +503,21 @@ __global__ void __launch_bounds__(LT_WARPS * 32) latent_attention_tc_kernel(
     // weighted latents: this warp's NTW * 8 columns
 #pragma unroll
     for (int kk = 0; kk < LT_BK / 16; ++kk) {
-      uint32_t a[2][4];
-      lt_ldsm4(a[0], Ps + (size_t)(lane & 15) * (LT_BK + 8) + kk * 16 + (lane >> 4) * 8);
-      lt_ldsm4(a[1], Ps + (size_t)(16 + (lane & 15)) * (LT_BK + 8) + kk * 16 + (lane >> 4) * 8);
+      uint32_t a[WT][2][4];
+#pragma unroll
+      for (int term = 0; term < WT; ++term) {
+        lt_ldsm4(a[term][0], Ps + term * PLANE + (size_t)(lane & 15) * (LT_BK + 8) + kk * 16 + (lane >> 4) * 8);
+        lt_ldsm4(a[term][1], Ps + term * PLANE + (size_t)(16 + (lane & 15)) * (LT_BK + 8) + kk * 16 + (lane >> 4) * 8);
+      }
 #pragma unroll
       for (int nt = 0; nt < NTW; ++nt) {
         uint32_t b[2];
         lt_ldsm2t(b, Kb + (size_t)(kk * 16 + (lane & 15)) * ldk + (warp * NTW + nt) * 8);
-        lt_mma(o[0][nt], a[0], b);
-        lt_mma(o[1][nt], a[1], b);
+#pragma unroll
+        for (int term = WT - 1; term >= 0; --term) {         // the small terms first
+          lt_mma(o[0][nt], a[term][0], b);
+          lt_mma(o[1][nt], a[term][1], b);
+        }
       }
     }
     __syncthreads();
@@ -519,15 +537,18 @@ __global__ void __launch_bounds__(LT_WARPS * 32) latent_attention_tc_kernel(
     }
 }
 
-// lat[row][:] (bfloat16) = the partial results of a (token, head) row merged: sum_s e^(m_s - M) o_s / sum_s e^(m_s - M) l_s
+// lat[row][:] (bfloat16) = the partial results of a (token, head) row merged: sum_s e^(m_s - M) o_s / (sum_s e^(m_s - M) l_s +
+// e^(sink[head] - M) where there are sinks)
 __global__ void __launch_bounds__(128) latent_merge_kernel(bf16* __restrict__ lat, const float* __restrict__ part_o,
-                                                           const float* __restrict__ part_ml, int rank, int splits, int total_rows) {
+                                                           const float* __restrict__ part_ml, int rank, int splits, int total_rows,
+                                                           const float* __restrict__ sink, int H) {
   pdl_wait();
   pdl_launch_dependents();
   const size_t row = blockIdx.x;
-  float M = -INFINITY;
+  const float sk = sink ? sink[row % H] : -INFINITY;
+  float M = sk;
   for (int s = 0; s < splits; ++s) M = fmaxf(M, part_ml[2 * ((size_t)s * total_rows + row)]);
-  float L = 0.f;
+  float L = sink ? expf(sk - M) : 0.f;
   for (int s = 0; s < splits; ++s) {
     const float m = part_ml[2 * ((size_t)s * total_rows + row)];
     if (m != -INFINITY) L += expf(m - M) * part_ml[2 * ((size_t)s * total_rows + row) + 1];
@@ -552,21 +573,24 @@ extern "C" long long qv_latent_tc_workspace_bytes(int T, int H, int dr, int rank
   return rows * (rank + dr) * 2 + (long long)splits * rows * rank * 4 + (long long)splits * rows * 2 * 4 + rows * rank * 2 + 64;
 }
 
+// weight_terms: see the kernel; sink: one number per head, or null.
 // bfloat16 operands; rank a multiple of 64 up to 512 (not 320 or 448), dr a multiple of 16, dn a multiple of 8.
 // wuk_t: the heads' key matrices transposed, [H][rank][dn].  workspace: what qv_latent_tc_workspace_bytes says,
 // 16-byte aligned.  Refuses other sizes (the caller then takes the generic kernel).
 extern "C" int qv_latent_attention_tc(void* out, int ld_out, const void* q, int ld_q, const void* gate, int ld_gate, const void* cache,
                                       const void* wuk_t, const void* wuv, const int* seg_q_start, const int* seg_pos0,
                                       const int* block_table, int max_blocks, int T, int S, int max_q_len, int H, int dn, int dr,
-                                      int dv, int rank, int page, int window, float scale, int splits, void* workspace, void* stream) {
+                                      int dv, int rank, int page, int window, float scale, int splits, void* workspace,
+                                      const float* sink, int weight_terms, void* stream) {
   if (T <= 0) return 0;
   if (rank % 64 || rank > 512 || dr % 16 || dr < 0 || dn % 8 || dn <= 0 || ld_q % 8 || splits < 1 || S > 65535 || splits > 65535 || H > 65535)
     return QV_ERR_UNSUPPORTED;
   if ((T + 63) / 64 > 65535) return QV_ERR_TOO_LARGE;
+  if (weight_terms != 1 && weight_terms != 3) return QV_ERR_UNSUPPORTED;
   const int ntw = rank / 64;
   if (ntw == 5 || ntw == 7) return QV_ERR_UNSUPPORTED;
   const int kw = rank + dr, ldk = kw + 8;
-  const size_t smem = ((size_t)LT_BM * ldk + (size_t)2 * LT_BK * ldk + (size_t)LT_BM * (LT_BK + 8)) * 2 + (size_t)2 * LT_WARPS * LT_BM * 4;
+  const size_t smem = ((size_t)LT_BM * ldk + (size_t)2 * LT_BK * ldk + (size_t)weight_terms * LT_BM * (LT_BK + 8)) * 2 + (size_t)2 * LT_WARPS * LT_BM * 4;
   if (smem > 220 * 1024) return QV_ERR_UNSUPPORTED;
   cudaStream_t st = (cudaStream_t)stream;
   const long long rows = (long long)T * H;
@@ -579,21 +603,27 @@ extern "C" int qv_latent_attention_tc(void* out, int ld_out, const void* q, int 
                      (const bf16*)q, ld_q, dn + dr, (const bf16*)wuk_t, (const bf16*)nullptr, 0, 0, T, rank, dn, dr);
   if (rc) return rc;
   dim3 grid(((size_t)max_q_len * H + LT_BM - 1) / LT_BM, S, splits);
-#define LT_LAUNCH(N)                                                                                                        \
-  case N:                                                                                                                   \
-    cudaFuncSetAttribute(latent_attention_tc_kernel<N>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);            \
-    rc = qv_launch(latent_attention_tc_kernel<N>, grid, dim3(LT_WARPS * 32), smem, st, part_o, part_ml, (const bf16*)qlat,  \
+#define LT_LAUNCH_WT(N, W)                                                                                                  \
+  do {                                                                                                                      \
+    cudaFuncSetAttribute(latent_attention_tc_kernel<N, W>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);         \
+    rc = qv_launch(latent_attention_tc_kernel<N, W>, grid, dim3(LT_WARPS * 32), smem, st, part_o, part_ml, (const bf16*)qlat, \
                    (const bf16*)cache, seg_q_start, seg_pos0, block_table, max_blocks, H, dr, page, window, scale, splits,  \
                    (int)rows);                                                                                              \
+  } while (0)
+#define LT_LAUNCH(N)                                               \
+  case N:                                                          \
+    if (weight_terms == 3) LT_LAUNCH_WT(N, 3);                     \
+    else LT_LAUNCH_WT(N, 1);                                       \
     break;
   switch (ntw) {
     LT_LAUNCH(1) LT_LAUNCH(2) LT_LAUNCH(3) LT_LAUNCH(4) LT_LAUNCH(6) LT_LAUNCH(8)
     default: return QV_ERR_UNSUPPORTED;
   }
 #undef LT_LAUNCH
+#undef LT_LAUNCH_WT
   if (rc) return rc;
   rc = qv_launch(latent_merge_kernel, dim3((unsigned)rows), dim3(128), 0, st, lat, (const float*)part_o, (const float*)part_ml, rank,
-                 splits, (int)rows);
+                 splits, (int)rows, sink, H);
   if (rc) return rc;
   // the heads' value matrices and the gate: per head latent [T, rank] x Wuv_h^T [rank, dv]
   if (gate)

@@ -4,7 +4,10 @@
 // qv_moe_route    logits = Wr h in float32 (fixed summation order), the `top` largest per token (ties: the lower
 //                 index), weights = softmax over the chosen logits only; optionally one more row of the router
 //                 matrix' companion (a scalar gate per token: sigmoid(ws . h)).  With `correction`: scores = softmax over all
-//                 logits, the choice by score + correction, weights = scores * w_scale (not renormalised).
+//                 logits, the choice by score + correction, weights = scores * w_scale (not renormalised).  In sigmoid mode:
+//                 scores = sigmoid(logits), the choice by score + correction among the experts of the `keep` best of `groups`
+//                 equal groups of neighbours (a group counts the sum of its two largest choice scores), weights = the chosen
+//                 scores over their sum (+ 1e-20), times w_scale.
 // qv_moe_route_table  no router: row `token id` of an integer table [vocab, top] lists the token's experts, each weighted 1/top.
 // qv_moe_group    counting sort of the (token, choice) pairs by expert, all on the device (a step never waits
 //                 for the host): row_token[r] = token of sorted row r, slot_row[token * top + j] = its sorted row,
@@ -172,7 +175,8 @@ template <typename T, typename TW>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(int* __restrict__ top_idx, float* __restrict__ top_w, float* __restrict__ gate_out,
                                                         const T* __restrict__ h, int ld_h, const TW* __restrict__ wr,
                                                         const TW* __restrict__ wg, int d, int E, int top, const float* __restrict__ pre,
-                                                        const float* __restrict__ correction, float w_scale) {
+                                                        const float* __restrict__ correction, float w_scale, int sigmoid, int groups,
+                                                        int keep) {
   extern __shared__ float logit[];           // E floats, then the token's d inputs
   pdl_wait();
   pdl_launch_dependents();
@@ -196,7 +200,34 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(int* __rest
   __syncthreads();
   if (warp != 0) return;
   float* score = xs + d;                     // E floats, with `correction`: the scores, while logit[] holds what the choice is by
-  if (correction) {
+  if (sigmoid) {
+    for (int e = lane; e < E; e += 32) {
+      score[e] = 1.0f / (1.0f + expf(-logit[e]));
+      logit[e] = score[e] + (correction ? correction[e] : 0.f);
+    }
+    __syncwarp();
+    if (keep < groups) {
+      float* gscore = score + E;             // one number per group
+      const int each = E / groups;
+      for (int g = lane; g < groups; g += 32) {
+        float a = -INFINITY, b = -INFINITY;  // the two largest of the group
+        for (int i = 0; i < each; ++i) {
+          const float v = logit[g * each + i];
+          if (v > a) { b = a; a = v; }
+          else if (v > b) b = v;
+        }
+        gscore[g] = each > 1 ? a + b : a;
+      }
+      __syncwarp();
+      for (int g = lane; g < groups; g += 32) {
+        int ahead = 0;                       // groups that come before this one (ties: the lower index)
+        for (int o = 0; o < groups; ++o) ahead += gscore[o] > gscore[g] || (gscore[o] == gscore[g] && o < g);
+        if (ahead >= keep)
+          for (int i = 0; i < each; ++i) logit[g * each + i] = -INFINITY;
+      }
+      __syncwarp();
+    }
+  } else if (correction) {
     float mx = -INFINITY, sum = 0.f;
     for (int e = lane; e < E; e += 32) mx = fmaxf(mx, logit[e]);
     mx = warp_max(mx);
@@ -212,7 +243,7 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(int* __rest
     }
     __syncwarp();
   }
-  float first = 0.f, denom = 0.f;
+  float first = 0.f, denom = 0.f, chosen = 0.f;
   for (int j = 0; j < top; ++j) {
     float best = -INFINITY;
     int bi = 0x7fffffff;
@@ -229,9 +260,11 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(int* __rest
     if (j == 0) first = best;
     const float p = expf(best - first);         // the first choice is the largest: exponents are <= 0
     denom += p;
-    if (lane == 0 && correction) {
+    if (lane == 0 && (correction || sigmoid)) {
+      const float sv = score[bi < E ? bi : 0];
       top_idx[(size_t)t * top + j] = bi < E ? bi : 0;
-      top_w[(size_t)t * top + j] = score[bi < E ? bi : 0] * w_scale;
+      top_w[(size_t)t * top + j] = sigmoid ? sv : sv * w_scale;
+      chosen += sv;
       if (bi < E) logit[bi] = -INFINITY;
     } else if (lane == 0) {
       top_idx[(size_t)t * top + j] = bi < E ? bi : 0;          // (not-a-number logits: still an expert that exists)
@@ -239,6 +272,11 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(int* __rest
       if (bi < E) logit[bi] = -INFINITY;
     }
     __syncwarp();
+  }
+  if (sigmoid) {
+    chosen = __shfl_sync(0xffffffffu, chosen, 0);
+    for (int j = lane; j < top; j += 32) top_w[(size_t)t * top + j] = top_w[(size_t)t * top + j] / (chosen + 1e-20f) * w_scale;
+    return;
   }
   if (correction) return;
   for (int j = lane; j < top; j += 32) top_w[(size_t)t * top + j] /= denom;
@@ -249,11 +287,12 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_kernel(int* __rest
 // result is the same whichever kernel forms them (same sums, same order).
 extern "C" int qv_moe_route(int* top_idx, float* top_w, float* gate_out, const void* h, int ld_h, const void* wr, const void* wg,
                             float* logits_ws, int T, int d, int E, int top, int dt, int w_dt, const float* correction, float w_scale,
-                            void* stream) {
+                            int sigmoid, int groups, int keep, void* stream) {
   if (T <= 0) return 0;
   if (E <= 0 || top <= 0 || top > E || E > 8192) return QV_ERR_UNSUPPORTED;
+  if (groups < 1 || keep < 1 || keep > groups || E % groups || top > keep * (E / groups) || (groups > 1 && !sigmoid)) return QV_ERR_UNSUPPORTED;
   cudaStream_t st = (cudaStream_t)stream;
-  const size_t smem = (size_t)(E + d + (correction ? E : 0)) * sizeof(float);
+  const size_t smem = (size_t)(E + d + (correction || sigmoid ? E : 0) + (keep < groups ? groups : 0)) * sizeof(float);
   if (smem > 48 * 1024) return QV_ERR_TOO_LARGE;
   const bool split = logits_ws && T <= 256;
   // more tokens: the logits by groups of tokens, where the group's rows fit shared memory
@@ -276,7 +315,7 @@ extern "C" int qv_moe_route(int* top_idx, float* top_w, float* gate_out, const v
     }                                                                                                                        \
     return qv_launch(moe_route_kernel<TT, TW>, dim3(T), dim3(ROUTE_WARPS * 32), smem, st, top_idx, top_w, gate_out, (const TT*)h, \
                      ld_h, (const TW*)wr, (const TW*)wg, d, E, top,                                                          \
-                     (split || tokens) ? (const float*)logits_ws : (const float*)nullptr, correction, w_scale);              \
+                     (split || tokens) ? (const float*)logits_ws : (const float*)nullptr, correction, w_scale, sigmoid, groups, keep); \
   } while (0)
   if (dt == QV_DT_F32 && w_dt == QV_DT_F32) ROUTE(float, float);
   if (dt == QV_DT_BF16 && w_dt == QV_DT_BF16) ROUTE(bf16, bf16);

@@ -60,14 +60,14 @@ _ARGTYPES = {
     "qv_sum2": [_V, _V, _V, _L, _I, _I, _V],
     "qv_softcap": [_V, _L, _F, _V],
     "qv_latent_prepare": [_V, _I, _V, _I, _I, _V, _V, _F, _V, _I, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _V],
-    "qv_latent_attention_generic": [_V, _I, _V, _I, _V, _I, _V, _V, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _V],
+    "qv_latent_attention_generic": [_V, _I, _V, _I, _V, _I, _V, _V, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _V, _V],
     "qv_latent_tc_workspace_bytes": [_I, _I, _I, _I, _I],
-    "qv_latent_attention_tc": [_V, _I, _V, _I, _V, _I, _V, _V, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _V, _V],
+    "qv_latent_attention_tc": [_V, _I, _V, _I, _V, _I, _V, _V, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _V, _V, _I, _V],
     "qv_conv_state": [_V, _I, _V, _I, _V, _V, _V, _L, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _V],
     "qv_linear_scan_state_floats": [_I, _I, _I, _I],
     "qv_linear_scan": [_I, _V, _I, _V, _I, _I, _V, _I, _V, _I, _V, _I, _V, _I, _V, _V, _V, _F, _F, _V, _L, _V, _V, _I, _I, _I, _I, _I, _V],
     "qv_gated_group_norm": [_V, _I, _V, _I, _V, _I, _V, _I, _I, _I, _F, _I, _I, _V],
-    "qv_moe_route": [_V, _V, _V, _V, _I, _V, _V, _V, _I, _I, _I, _I, _I, _I, _V, _F, _V],
+    "qv_moe_route": [_V, _V, _V, _V, _I, _V, _V, _V, _I, _I, _I, _I, _I, _I, _V, _F, _I, _I, _I, _V],
     "qv_moe_max_tiles": [_I, _I, _I],
     "qv_moe_tile_rows": [_I],
     "qv_moe_group": [_V, _V, _V, _V, _V, _I, _I, _I, _I, _V],
@@ -78,7 +78,9 @@ _ARGTYPES = {
     "qv_scale_sum2": [_V, _V, _V, _V, _V, _I, _I, _I, _I, _V],
     "qv_stream_concat": [_V, _V, _V, _V, _I, _I, _I, _I, _V],
     "qv_add_vector": [_V, _V, _I, _I, _V],
-    "qv_activation": [_V, _V, _L, _I, _I, _V],
+    "qv_activation": [_V, _V, _V, _L, _I, _I, _I, _V],
+    "qv_stream_pass": [_V, _V, _V, _V, _I, _V, _V, _V, _V, _F, _V, _I, _I, _I, _I, _I, _I, _V],
+    "qv_cache_rows": [_V, _V, _I, _V, _V, _V, _I, _I, _I, _I, _I, _V],
     "qv_diff_prepare": [_V, _I, _V, _I, _V, _V, _V, _F, _V, _I, _V, _V, _V, _I, _V, _I, _I, _I, _I, _I, _I, _I, _I, _I, _V],
     "qv_diff_partial_floats": [_I],
     "qv_diff_attention_tc": [_V, _I, _V, _I, _V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _V, _I, _V],
@@ -347,11 +349,57 @@ def add_vector(x, v) -> None:
 ACT_RELU2, ACT_GELU_TANH = 0, 1
 
 
-def activation(out, x, kind: int = ACT_RELU2) -> None:
-    """out = act(x) elementwise (out may be x); kind ACT_RELU2: the square of relu, ACT_GELU_TANH: the tanh form of GELU."""
-    _need_cuda(out, x)
+def activation(out, x, kind: int = ACT_RELU2, bias=None) -> None:
+    """out = act(x + bias) elementwise (out may be x; bias float32, one per column, or None); kind ACT_RELU2: the square of relu,
+    ACT_GELU_TANH: the tanh form of GELU."""
+    _need_cuda(out, x, bias)
     assert out.dtype == x.dtype and out.is_contiguous() and x.is_contiguous() and out.numel() == x.numel()
-    _check(_lib("elementwise").qv_activation(_ptr(out), _ptr(x), x.numel(), kind, dt_code(x.dtype), _stream()), "activation")
+    assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == x.shape[-1])
+    _check(_lib("elementwise").qv_activation(_ptr(out), _ptr(x), _ptr(bias), x.numel(), x.shape[-1], kind, dt_code(x.dtype), _stream()), "activation")
+
+
+MAX_STREAMS = 16
+
+
+def stream_pass(out, streams, read_coef, weight=None, eps: float = 0.0, y=None, y_bias=None, write_coef=None, x0=None, row_idx=None,
+                store: bool = True) -> None:
+    """One pass over several residual streams (streams [T, S, d] float32): the write that is pending and the next read.
+    With write_coef (float32, [S * S mix from/to, then S out]): x_t <- sum_s mix[s, t] x_s + out[t] * (y + y_bias); the old streams are
+    those of `streams`, or x0 [T, d] for all of them; with `store` the new ones go to `streams`.  out = sum_s read_coef[s] x_s, or,
+    with weight (float32 [d]), its RMS norm times weight.  row_idx: the tokens whose rows are read (nothing is stored then)."""
+    _need_cuda(out, streams, read_coef, weight, y, y_bias, write_coef, x0, row_idx)
+    T, S, d = streams.shape
+    rows = out.shape[0]
+    assert streams.dtype == torch.float32 and streams.is_contiguous() and out.is_contiguous() and out.shape[1] == d
+    assert read_coef.dtype == torch.float32 and read_coef.is_contiguous() and read_coef.numel() == S
+    assert weight is None or (weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == d)
+    assert x0 is None or (x0.dtype == torch.float32 and x0.is_contiguous() and tuple(x0.shape) == (T, d))
+    if write_coef is not None:
+        assert write_coef.dtype == torch.float32 and write_coef.is_contiguous() and write_coef.numel() == S * S + S
+        assert tuple(y.shape) == (T, d) and y.stride(1) == 1
+        assert y_bias is None or (y_bias.dtype == torch.float32 and y_bias.is_contiguous() and y_bias.numel() == d)
+    if row_idx is not None:
+        _i32(row_idx, "row_idx")
+        assert row_idx.numel() >= rows
+        store = False
+    else:
+        assert rows == T
+    rc = _lib("elementwise").qv_stream_pass(
+        _ptr(out), _ptr(streams), _ptr(x0), _ptr(y), y.stride(0) if y is not None else 0, _ptr(y_bias), _ptr(write_coef), _ptr(read_coef),
+        _ptr(weight), float(eps), _ptr(row_idx), rows, S, d, 1 if store else 0, dt_code(y.dtype) if y is not None else dt_code(out.dtype),
+        dt_code(out.dtype), _stream())
+    _check(rc, "stream_pass")
+
+
+def cache_rows(cache_layer, src, ctx, block_table, page: int) -> None:
+    """The token's row of cache_layer [pages, page, width] = src[t] (columns of a wider tensor are fine; equal types)."""
+    _need_cuda(cache_layer, src, block_table)
+    T, width = src.shape
+    assert src.stride(1) == 1 and src.dtype == cache_layer.dtype and cache_layer.is_contiguous() and tuple(cache_layer.shape[1:]) == (page, width)
+    _i32(block_table, "block_table")
+    rc = _lib("elementwise").qv_cache_rows(_ptr(cache_layer), _ptr(src), src.stride(0), _ptr(ctx.tok_pos), _ptr(ctx.tok_seg), _ptr(block_table),
+                                           block_table.shape[-1], T, width, page, dt_code(src.dtype), _stream())
+    _check(rc, "cache_rows")
 
 
 def add_tanhnorm(out, residual, delta, weight, bias, alpha: float, row_idx=None) -> None:
@@ -456,14 +504,15 @@ def rmsnorm_rows(out, x, weight, eps: float) -> None:
 # ------------------------------------------------------------------ differential attention
 
 def diff_prepare(q_out, proj, bias, q_weight, k_weight, eps, cos_sin, ctx, block_table, cache_layer, H, G, n, dv, rot, page) -> None:
-    """Per token of proj (float32 or the compute type; columns [q: H*2n | k: G*2n | v: G*dv]): bias added, every map of q and
-    k RMS-normed over n with its weight and rotated over its first `rot` entries (pairs i, i + rot/2); q -> q_out [T, H*2n],
+    """Per token of proj (float32 or the compute type; columns [q: H*2n | k: G*2n | v: G*dv]): bias (or None) added, every map of q
+    and k RMS-normed over n with its weight (q_weight and k_weight None: not normed) and rotated over its first `rot` entries (pairs i, i + rot/2); q -> q_out [T, H*2n],
     k and v -> the token's row of cache_layer [pages, page, G*(2n+dv)]."""
     _need_cuda(q_out, proj, bias, q_weight, k_weight, cos_sin, block_table, cache_layer)
     T = proj.shape[0]
     assert proj.stride(1) == 1 and proj.shape[1] == (H + G) * 2 * n + G * dv and q_out.stride(1) == 1 and q_out.shape == (T, H * 2 * n)
     assert cache_layer.is_contiguous() and tuple(cache_layer.shape[1:]) == (page, G * (2 * n + dv)) and cache_layer.dtype == q_out.dtype
-    assert q_weight.dtype == k_weight.dtype == torch.float32 and q_weight.numel() == k_weight.numel() == n
+    assert (q_weight is None) == (k_weight is None)
+    assert q_weight is None or (q_weight.dtype == k_weight.dtype == torch.float32 and q_weight.numel() == k_weight.numel() == n)
     assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == proj.shape[1])
     if rot:
         assert cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and cos_sin.shape[1] * 2 == rot
@@ -558,23 +607,24 @@ def latent_prepare(proj, q, kv_off: int, cache_layer, norm_w, eps, cos_sin, ctx,
     """Per token of proj (rows [.. down: rank+dr at kv_off ..]): the latent part of the down projection RMS-normed, the
     shared key part rotated (pairs 2i, 2i+1, or i, i + rot/2 with split_half), both written to the token's row of
     cache_layer [pages, page, rank+dr]; every head's rotated query part of q [T, H*(dn+dr)] (columns of proj or a tensor
-    of its own) rotated in place."""
+    of its own) rotated in place.  rot 0: nothing is rotated (cos_sin None)."""
     _need_cuda(proj, q, cache_layer, norm_w, cos_sin, block_table)
     assert proj.stride(1) == 1 and cache_layer.is_contiguous() and cache_layer.dtype == proj.dtype == q.dtype
     assert q.stride(1) == 1 and q.shape[0] == proj.shape[0] and q.shape[1] == H * (dn + dr)
     assert tuple(cache_layer.shape[1:]) == (page, rank + dr) and norm_w.dtype == torch.float32 and norm_w.numel() == rank
-    assert cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and cos_sin.shape[1] * 2 == rot
+    assert (rot == 0) if cos_sin is None else (cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and cos_sin.shape[1] * 2 == rot)
     _i32(block_table, "block_table")
     rc = _lib("latent_attention").qv_latent_prepare(
-        _ptr(proj), proj.stride(0), _ptr(q), q.stride(0), kv_off, _ptr(cache_layer), _ptr(norm_w), eps, _ptr(cos_sin), cos_sin.shape[0],
+        _ptr(proj), proj.stride(0), _ptr(q), q.stride(0), kv_off, _ptr(cache_layer), _ptr(norm_w), eps, _ptr(cos_sin),
+        cos_sin.shape[0] if cos_sin is not None else 1,
         _ptr(ctx.tok_pos), _ptr(ctx.tok_seg), _ptr(block_table), block_table.shape[-1], proj.shape[0], H, dn, dr, rank, rot, page,
         1 if split_half else 0, dt_code(proj.dtype), _stream())
     _check(rc, "latent_prepare")
 
 
-def latent_attention_generic(out, q, gate, cache_layer, wuk, wuv, ctx, block_table, H, dn, dr, dv, rank, page, window, scale) -> None:
+def latent_attention_generic(out, q, gate, cache_layer, wuk, wuv, ctx, block_table, H, dn, dr, dv, rank, page, window, scale, sink=None) -> None:
     """out[t, h*dv:(h+1)*dv] = gate * Wuv_h (softmax-weighted latent) for every token and head, the query carried
-    into the latent space by Wuk_h; float32 arithmetic, any sizes.  q: [T, H*(dn+dr)] (a column slice is fine)."""
+    into the latent space by Wuk_h; with sink (float32 [H]) exp(sink[h]) joins the softmax' denominator; float32 arithmetic, any sizes.  q: [T, H*(dn+dr)] (a column slice is fine)."""
     _need_cuda(out, q, gate, cache_layer, wuk, wuv, block_table)
     assert q.stride(1) == 1 and out.stride(1) == 1 and q.dtype == out.dtype == cache_layer.dtype
     assert cache_layer.is_contiguous() and tuple(cache_layer.shape[1:]) == (page, rank + dr)
@@ -586,7 +636,7 @@ def latent_attention_generic(out, q, gate, cache_layer, wuk, wuv, ctx, block_tab
     rc = _lib("latent_attention").qv_latent_attention_generic(
         _ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(cache_layer),
         _ptr(wuk), _ptr(wuv), _ptr(ctx.tok_pos), _ptr(ctx.tok_seg), _ptr(block_table), block_table.shape[-1], q.shape[0], H, dn, dr,
-        dv, rank, page, window, scale, dt_code(q.dtype), dt_code(wuk.dtype), _stream())
+        dv, rank, page, window, scale, dt_code(q.dtype), dt_code(wuk.dtype), _ptr(_sinks(sink, H)), _stream())
     _check(rc, "latent_attention_generic")
 
 
@@ -598,10 +648,16 @@ def latent_attention_splits(ctx, H: int) -> int:
     return max(1, min(sm_count() // max(tiles, 1), blocks))
 
 
-def latent_attention_tc(out, q, gate, cache_layer, wuk_t, wuv, ctx, block_table, H, dn, dr, dv, rank, page, window, scale) -> bool:
+def _sinks(sink, H: int):
+    assert sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.is_cuda and sink.numel() == H)
+    return sink
+
+
+def latent_attention_tc(out, q, gate, cache_layer, wuk_t, wuv, ctx, block_table, H, dn, dr, dv, rank, page, window, scale, sink=None,
+                        weight_terms: int = 1) -> bool:
     """Latent attention on the tensor cores (bfloat16; rank a multiple of 64 up to 512, rotated part a multiple of 16,
-    unrotated part a multiple of 8).  wuk_t: the heads' key matrices transposed, [H, rank, dn].  False, nothing
-    written, for other sizes."""
+    unrotated part a multiple of 8).  wuk_t: the heads' key matrices transposed, [H, rank, dn].  weight_terms: how many bfloat16 terms a
+    softmax weight is split into for the product with the latents (3 hold its 24 bits).  False, nothing written, for other sizes."""
     if (q.dtype != torch.bfloat16 or wuk_t is None or wuk_t.dtype != torch.bfloat16 or wuv.dtype != torch.bfloat16 or rank % 64
             or rank > 512 or rank // 64 in (5, 7) or dr % 16 or dn % 8 or q.stride(0) % 8
             or (gate is not None and gate.dtype != torch.bfloat16)):
@@ -618,7 +674,8 @@ def latent_attention_tc(out, q, gate, cache_layer, wuk_t, wuv, ctx, block_table,
     rc = lib.qv_latent_attention_tc(
         _ptr(out), out.stride(0), _ptr(q), q.stride(0), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(cache_layer),
         _ptr(wuk_t), _ptr(wuv), _ptr(ctx.seg_q_start), _ptr(ctx.seg_pos0), _ptr(block_table), block_table.shape[-1], T,
-        ctx.num_segments, ctx.max_q_len, H, dn, dr, dv, rank, page, window, scale, splits, _ptr(ws), _stream())
+        ctx.num_segments, ctx.max_q_len, H, dn, dr, dv, rank, page, window, scale, splits, _ptr(ws), _ptr(_sinks(sink, H)), weight_terms,
+        _stream())
     if rc == -2:
         return False
     _check(rc, "latent_attention_tc")
@@ -626,13 +683,14 @@ def latent_attention_tc(out, q, gate, cache_layer, wuk_t, wuv, ctx, block_table,
     return True
 
 
-def latent_attention(out, q, gate, cache_layer, wuk, wuv, ctx, block_table, H, dn, dr, dv, rank, page, window, scale, wuk_t=None) -> None:
+def latent_attention(out, q, gate, cache_layer, wuk, wuv, ctx, block_table, H, dn, dr, dv, rank, page, window, scale, wuk_t=None, sink=None,
+                     weight_terms: int = 1) -> None:
     """Latent attention of every token of the step: the tensor-core kernels for bfloat16 where they take the sizes (and
     the transposed key matrices wuk_t [H, rank, dn] are given), else (and for float32) the CUDA-core kernel."""
     if q.dtype == torch.bfloat16 and latent_attention_tc(out, q, gate, cache_layer, wuk_t, wuv, ctx, block_table, H, dn, dr, dv, rank,
-                                                         page, window, scale):
+                                                         page, window, scale, sink=sink, weight_terms=weight_terms):
         return
-    latent_attention_generic(out, q, gate, cache_layer, wuk, wuv, ctx, block_table, H, dn, dr, dv, rank, page, window, scale)
+    latent_attention_generic(out, q, gate, cache_layer, wuk, wuv, ctx, block_table, H, dn, dr, dv, rank, page, window, scale, sink=sink)
 
 
 # ------------------------------------------------------------------ recurrent mixers
@@ -1050,11 +1108,14 @@ def head_delta_scan(out, qn, kn, v, coef, state, ctx, H: int, G: int, dk: int, d
 
 # ------------------------------------------------------------------ routed feed-forward
 
-def moe_route(top_idx, top_w, gate_out, h, w_router, w_gate, correction=None, w_scale: float = 1.0) -> None:
+def moe_route(top_idx, top_w, gate_out, h, w_router, w_gate, correction=None, w_scale: float = 1.0, sigmoid: bool = False, groups: int = 1,
+              keep: int = 1) -> None:
     """Per token: router logits in float32, the top choices (top_idx int32 [T, top]) and their weights (softmax
     over the chosen logits, top_w float32 [T, top]); gate_out [T] = sigmoid(w_gate . h) when w_gate is given.  With
     `correction` (float32, a number per row of the router): scores are the softmax over all logits, the choice goes by
-    score + correction and the weights are the chosen scores times w_scale."""
+    score + correction and the weights are the chosen scores times w_scale.  With `sigmoid`: scores are the sigmoids of the logits,
+    the choice goes by score + correction within the `keep` best of `groups` equal groups of neighbours (a group counts the sum of
+    its two largest choice scores), and the weights are the chosen scores over their sum, times w_scale."""
     _need_cuda(top_idx, top_w, gate_out, h, w_router, w_gate, correction)
     assert correction is None or (correction.dtype == torch.float32 and correction.is_contiguous() and correction.numel() == w_router.shape[0])
     T, d = h.shape
@@ -1065,7 +1126,7 @@ def moe_route(top_idx, top_w, gate_out, h, w_router, w_gate, correction=None, w_
     ws = torch.empty(T * (E + 1), device=h.device, dtype=torch.float32) if few else None
     rc = _lib("moe").qv_moe_route(_ptr(top_idx), _ptr(top_w), _ptr(gate_out), _ptr(h), h.stride(0), _ptr(w_router), _ptr(w_gate),
                                   _ptr(ws), T, d, E, top, dt_code(h.dtype), dt_code(w_router.dtype), _ptr(correction), float(w_scale),
-                                  _stream())
+                                  1 if sigmoid else 0, int(groups), int(keep), _stream())
     _check(rc, "moe_route")
     if few:
         add_launches(1)

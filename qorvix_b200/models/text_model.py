@@ -34,6 +34,12 @@ class TextModel:
         self.loop = build_part("stream", getattr(spec, "loop", None), source, rt)
         # the stream after each run as a weighted sum of all runs' results (None: the run's result as it is)
         self.depth = build_part("stream", getattr(spec, "depth_average", None), source, rt)
+        # the residual as several streams (None: one)
+        self.streams = build_part("stream", getattr(spec, "streams", None), source, rt)
+        if any(getattr(b, "takes_streams", False) != (self.streams is not None) for b in self.blocks):
+            raise ValueError("blocks for several residual streams and blocks for one do not go together")
+        if self.streams is not None and (self.loop is not None or self.depth is not None):
+            raise ValueError("a loop's re-entry and a depth average work on one residual stream")
         self._more_views = {}          # run -> the indices of the further caches of a mixer that keeps several
         self.stream_tap = None         # callable(run, residual, pending) after every run: for tests and debugging
         self._native = None            # the native executor of this model over a cache, made on first use (False: not applicable)
@@ -92,6 +98,8 @@ class TextModel:
         else:
             ops.embed(residual, self.embedding, ctx.token_ids)
         pending = None
+        if self.streams is not None:               # residual: [T, streams, width] from here on, pending: a StreamDelta
+            residual, pending = self.streams.begin(residual)
         x0 = None
         if self.loop is not None:                  # the embedding's output, kept for the passes' re-entries
             x0 = torch.empty_like(residual)
@@ -110,10 +118,16 @@ class TextModel:
             if self.depth is not None:
                 residual, pending = self.depth.after(run, residual, pending, stack), None
             if self.stream_tap is not None:
-                self.stream_tap(run, residual, pending)
+                if self.streams is not None:
+                    self.stream_tap(run, self.streams.total(residual, pending), None)
+                else:
+                    self.stream_tap(run, residual, pending)
         if ctx.num_wanted == 0:
             return None
-        h = self.final_norm.add_norm(residual, pending, rows=ctx.want_rows)
+        if self.streams is not None:
+            h = self.streams.final(self.final_norm, residual, pending, ctx.want_rows)
+        else:
+            h = self.final_norm.add_norm(residual, pending, rows=ctx.want_rows)
         logits = self.lm_head(h, out_dtype=torch.float32)
         if self.spec.logit_softcap:
             ops.softcap(logits, self.spec.logit_softcap)
@@ -133,3 +147,4 @@ class _BlockView:
         self.residual_mult = getattr(layer, "residual_mult", 1.0)
         self.mixer_gate, self.ffn_gate = getattr(layer, "mixer_gate", None), getattr(layer, "ffn_gate", None)
         self.mixer_post_norm, self.ffn_post_norm = getattr(layer, "mixer_post_norm", None), getattr(layer, "ffn_post_norm", None)
+        self.mixer_link, self.ffn_link = getattr(layer, "mixer_link", None), getattr(layer, "ffn_link", None)

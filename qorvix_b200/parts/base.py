@@ -4,6 +4,8 @@ Mixer         forward(x[T,d], ctx, cache) -> [T,d] in the compute dtype; cache_s
               it keeps per request (cache.spec.PagedKVSpec / FixedStateSpec / None);
               reads_cache_of() names another layer whose cache it reads instead.
 FeedForward   forward(x[T,d], ctx) -> [T,d].
+              One whose last product has a bias may offer it as output_bias and take with_bias=False: a
+              block then adds it in the pass that takes the output.
               A mixer or feed-forward with the attribute folds_norms = True also takes x as a
               PreNormed and the keywords residual=<float32 stream>, next_norm=<the RMS norm that reads
               the stream next>; it may then add its output to the stream itself and return a
@@ -22,7 +24,8 @@ Position      table() -> float32 [positions, rotary_dim/2, 2] of (cos, sin) if i
               in place for mixers that do not fuse it.
 Block         forward(residual, pending, ctx, cache) -> (residual, pending): `pending` is a
               delta not yet added to the residual stream, so that the next norm adds it in
-              the same pass.
+              the same pass.  A block with takes_streams = True has the residual as several streams
+              [T, streams, d] and a StreamDelta as pending (parts/streams.py).
 """
 from __future__ import annotations
 
@@ -76,6 +79,17 @@ class ReadyNormed(PreNormed):
         return self.rows
 
 
+@dataclass
+class StreamDelta:
+    """What is pending where the residual is several streams (parts/streams.py): a sublayer's output `y` (plus `bias`) that has yet
+    to go back by its `link`, and, ahead of the first store, the one row x0 that all streams still equal (the stream
+    tensor then holds nothing)."""
+    link: object = None
+    y: Optional[torch.Tensor] = None
+    bias: Optional[torch.Tensor] = None
+    x0: Optional[torch.Tensor] = None
+
+
 class Mixer:
     def cache_spec(self):
         return None
@@ -111,5 +125,7 @@ class PositionEncoding:
 
 
 class Block:
+    takes_streams = False              # True: the residual is several streams
+
     def forward(self, residual, pending, ctx, cache):
         raise NotImplementedError

@@ -2,7 +2,7 @@
     x += mixer(norm(x));  x += feed_forward(norm(x))
 The residual stream is float32.  A block hands the feed-forward's output on as a pending
 delta, which the next norm adds in its own pass.  'post_norm' puts the norms on the parts' outputs instead, 'sandwich_norm'
-on both sides of a part."""
+on both sides of a part; 'hyper' is 'pre_norm' over several residual streams."""
 from __future__ import annotations
 
 import torch
@@ -11,6 +11,7 @@ from ..csrc import ops
 from .base import Block, PreNormed, ReadyNormed
 from .linear import Linear
 from .registry import build_part, register_part
+from .streams import StreamLink
 
 
 class PreNormBlock(Block):
@@ -273,6 +274,38 @@ class SandwichNormBlock(Block):
         return self.mixer_norm if self.mixer is not None else self.ffn_norm
 
 
+class HyperBlock(Block):
+    """The pre-norm order on several residual streams (parts/streams.py): each part reads the normed weighted sum of the streams and
+    its output goes back to all of them in the pass in which the next part reads."""
+    takes_streams = True
+
+    def __init__(self, spec, source, rt):
+        self.rt = rt
+        self.mixer = build_part("mixer", spec.mixer, source, rt)
+        self.feed_forward = build_part("feed_forward", spec.feed_forward, source, rt)
+        self.mixer_norm = build_part("norm", spec.mixer_norm, source, rt) if self.mixer is not None else None
+        self.ffn_norm = build_part("norm", spec.ffn_norm, source, rt) if self.feed_forward is not None else None
+        mult = float(getattr(spec, "residual_mult", 1.0))
+        self.mixer_link = StreamLink(spec.mixer_link, mult, source, rt) if self.mixer is not None else None
+        self.ffn_link = StreamLink(spec.ffn_link, mult, source, rt) if self.feed_forward is not None else None
+
+    def forward(self, streams, pending, ctx, cache):
+        if self.mixer is not None:
+            x, left = self.mixer_link.read(streams, pending, self.mixer_norm)
+            pending = self.mixer_link.deliver(self.mixer.forward(x, ctx, cache), left)
+        ff = self.feed_forward
+        if ff is not None:
+            x, left = self.ffn_link.read(streams, pending, self.ffn_norm)
+            bias = getattr(ff, "output_bias", None)
+            y = ff.forward(x, ctx) if bias is None else ff.forward(x, ctx, with_bias=False)
+            pending = self.ffn_link.deliver(y, left, bias)
+        return streams, pending
+
+    def first_norm(self):
+        return None                              # the streams are summed ahead of it: nothing for the block ahead to prepare
+
+
+register_part("block", "hyper", HyperBlock)
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "sandwich_norm", SandwichNormBlock)
 register_part("block", "post_norm", PostNormBlock)

@@ -3,8 +3,8 @@ rotated key part shared by all heads are kept, in pages; a head's unrotated keys
 W_uk c and W_uv c.  The kernels never expand them: the query is carried into the latent space
 (W_uk^T q), attention runs over the cache rows as they are, and W_uv is applied to the weighted latent
 (csrc/latent_attention.cu).  Query, down projection and gate come from one fused product; a model whose queries pass a
-normed latent of their own has that latent's down matrix in the fused product and one more product behind the norm, and
-the gate may be absent."""
+normed latent of their own has that latent's down matrix in the fused product and one more product behind the norm; the gate
+and the rotated part may be absent, and a sink per head may take its share of the softmax."""
 from __future__ import annotations
 
 import torch
@@ -47,12 +47,16 @@ class LatentAttention(Mixer):
                        if self.k_up.dtype == torch.bfloat16 else None)
         self.o_proj = Linear(source.get(spec.o_proj))
         self.position = build_part("position", spec.position, source, rt)
+        self.sink = source.get(spec.sink, dtype=torch.float32) if getattr(spec, "sink", None) is not None else None
+        self.weight_terms = 3 if getattr(spec, "exact_weights", False) else 1
         pairing = getattr(spec.position, "pairing", "")
-        if pairing not in ("interleaved", "split_half") or self.position.table() is None:
+        if (self.position is None) != (self.dr == 0):
+            raise ValueError("latent attention: a rotated part needs a position encoding, and one without a rotated part has none")
+        if self.position is not None and (pairing not in ("interleaved", "split_half") or self.position.table() is None):
             raise ValueError("latent attention rotates pairs of entries from a cos/sin table: its position must be a rotary "
                              "encoding with pairing 'interleaved' or 'split_half'")
         self.split_half = pairing == "split_half"
-        self.rot = self.position.table().shape[1] * 2
+        self.rot = self.position.table().shape[1] * 2 if self.position is not None else 0
         self.window, self.scale, self.eps = int(spec.window), float(spec.scale), float(spec.eps)
 
     def cache_spec(self):
@@ -68,12 +72,12 @@ class LatentAttention(Mixer):
             q = self.q_up(cq, out_dtype=self.rt.dtype)
         else:
             q = proj[:, : self.kv_off]
-        ops.latent_prepare(proj, q, self.kv_off, cache.tensor, self.kv_norm, self.eps, self.position.table(), ctx, bt,
-                           H, dn, dr, rank, self.rot, cache.page_size, split_half=self.split_half)
+        ops.latent_prepare(proj, q, self.kv_off, cache.tensor, self.kv_norm, self.eps,
+                           self.position.table() if self.position is not None else None, ctx, bt, H, dn, dr, rank, self.rot, cache.page_size, split_half=self.split_half)
         gate = proj[:, self.gate_off: self.gate_off + H * dv] if self.gate_off is not None else None
         out = torch.empty((proj.shape[0], H * dv), device=proj.device, dtype=self.rt.dtype)
         ops.latent_attention(out, q, gate, cache.tensor, self.k_up, self.v_up, ctx, bt,
-                             H, dn, dr, dv, rank, cache.page_size, self.window, self.scale, wuk_t=self.k_up_t)
+                             H, dn, dr, dv, rank, cache.page_size, self.window, self.scale, wuk_t=self.k_up_t, sink=self.sink, weight_terms=self.weight_terms)
         return self.o_proj(out, out_dtype=self.rt.dtype)
 
 

@@ -68,7 +68,7 @@ class SwiGLU(FeedForward):
 
 class ActMLP(FeedForward):
     """Ungated feed-forward: down(act(up x)), the activation (the square of relu, or the tanh form of GELU) as a pass of
-    its own."""
+    its own, which also adds the up product's bias where there is one; the down product's bias is offered to the block."""
 
     def __init__(self, spec, source, rt):
         acts = {"relu2": ops.ACT_RELU2, "gelu_tanh": ops.ACT_GELU_TANH}
@@ -78,11 +78,18 @@ class ActMLP(FeedForward):
         self.rt = rt
         self.up = Linear(source.get(spec.up_proj))
         self.down = Linear(source.get(spec.down_proj))
+        bias = getattr(spec, "bias", False)
+        self.up_bias = source.get(spec.up_proj + ".b", dtype=torch.float32) if bias else None
+        self.output_bias = source.get(spec.down_proj + ".b", dtype=torch.float32) if bias else None
 
-    def forward(self, x, ctx):
+    def forward(self, x, ctx, with_bias: bool = True):
         act = self.up(x, out_dtype=self.rt.dtype)
-        ops.activation(act, act, self.act)
-        return self.down(act, out_dtype=self.rt.dtype)
+        ops.activation(act, act, self.act, bias=self.up_bias)
+        if self.output_bias is None or not with_bias:
+            return self.down(act, out_dtype=self.rt.dtype)
+        y = self.down(act, out_dtype=torch.float32)
+        ops.add_vector(y, self.output_bias)
+        return y
 
 
 register_part("feed_forward", "swiglu", SwiGLU)

@@ -34,6 +34,10 @@ class RoutedFeedForward(FeedForward):
         self.correction = source.get(spec.correction, dtype=torch.float32).reshape(-1).contiguous() if spec.correction is not None else None
         if spec.activation not in GLU_ACTIVATIONS:
             raise ValueError(f"unknown activation '{spec.activation}' (known: {', '.join(GLU_ACTIVATIONS)})")
+        if spec.scores not in ("softmax", "sigmoid"):
+            raise ValueError(f"unknown router scores '{spec.scores}' (known: softmax, sigmoid)")
+        self.routing = dict(correction=self.correction, w_scale=float(spec.route_scale), sigmoid=spec.scores == "sigmoid", groups=spec.groups,
+                            keep=spec.group_keep)
         self.glu = dict(act=GLU_ACTIVATIONS[spec.activation], limit=float(spec.limit), slope=float(spec.slope))
 
     def forward(self, x, ctx, add=None, add_scale=None, scale=None):
@@ -44,7 +48,7 @@ class RoutedFeedForward(FeedForward):
         top_idx = torch.empty((T, s.top), device=dev, dtype=torch.int32)
         top_w = torch.empty((T, s.top), device=dev, dtype=torch.float32)
         gate = torch.empty(T, device=dev, dtype=torch.float32) if self.shared_gate is not None else None
-        ops.moe_route(top_idx, top_w, gate, x, self.router, self.shared_gate, correction=self.correction, w_scale=s.route_scale)
+        ops.moe_route(top_idx, top_w, gate, x, self.router, self.shared_gate, **self.routing)
         tc = self.tensor_cores
         tile_rows = ops.moe_tile_rows(tc)
         ints = torch.empty(3 * R + 3 * ops.moe_max_tiles(R, s.experts, tile_rows), device=dev, dtype=torch.int32)

@@ -123,8 +123,8 @@ class BigramEmbeddingSpec:
 class LatentAttentionSpec:
     """Causal attention whose keys and values are expanded from a cached low-rank latent; each head's
     query and key have `head_dim` unrotated entries followed by `rot_dim` rotated ones, the rotated key
-    part being one vector shared by all heads; optionally a sigmoid gate multiplies the heads' outputs
-    (gate_proj), and optionally the queries pass a latent of their own: c = rmsnorm(q_down x) * q_norm,
+    part being one vector shared by all heads (rot_dim 0 with position None: nothing is rotated); optionally a sigmoid gate
+    multiplies the heads' outputs (gate_proj), optionally head h's softmax has exp(sink[h]) in its denominator, and optionally the queries pass a latent of their own: c = rmsnorm(q_down x) * q_norm,
     q = q_proj c with q_proj [heads * (head_dim + rot_dim), q_rank]."""
     hidden_size: int
     num_heads: int
@@ -134,7 +134,7 @@ class LatentAttentionSpec:
     kv_rank: int
     scale: float
     eps: float                    # of the latents' RMS norms
-    position: object              # RotarySpec over rot_dim; pairing 'interleaved' or 'split_half'
+    position: object              # RotarySpec over rot_dim; pairing 'interleaved' or 'split_half'; None where rot_dim is 0
     q_proj: str
     kv_down: str                  # [kv_rank + rot_dim, hidden]
     kv_norm: str
@@ -147,6 +147,8 @@ class LatentAttentionSpec:
     q_rank: int = 0               # > 0: the queries' latent size
     q_down: Optional[str] = None  # [q_rank, hidden]
     q_norm: Optional[str] = None  # [q_rank]
+    sink: Optional[str] = None    # [heads]
+    exact_weights: bool = False   # softmax weights enter the product with the latents with all their 24 bits (else rounded to the compute type)
 
     def tensors(self) -> TensorTable:
         H, d = self.num_heads, self.hidden_size
@@ -163,6 +165,8 @@ class LatentAttentionSpec:
             t[self.q_proj] = ((H * (self.head_dim + self.rot_dim), d), "matrix")
         if self.gate_proj is not None:
             t[self.gate_proj] = ((H * self.value_dim, d), "matrix")
+        if self.sink is not None:
+            t[self.sink] = ((H,), "normal:0:1")
         return t
 
 
@@ -244,7 +248,10 @@ class MoESpec:
     softmax over the chosen router logits; optionally a shared gated feed-forward for every token, scaled
     by the sigmoid of one number per token (shared_gate) or added as it is.
     With `correction` (a number per row of the router) scores are the softmax over ALL router logits, the choice goes by
-    score + correction and the weights are the chosen scores times route_scale.  The last `identity` rows of the router are
+    score + correction and the weights are the chosen scores times route_scale.
+    With scores 'sigmoid' they are the sigmoids of the logits, the choice goes by score + correction, and the weights are the
+    chosen scores over their sum, times route_scale; the experts may form `groups` equal groups of neighbours of which each
+    token's choice is limited to the group_keep best (a group counts the sum of its two largest choice scores).  The last `identity` rows of the router are
     identity experts: their output is the input itself, they have no matrices."""
     hidden_size: int
     experts: int
@@ -257,7 +264,10 @@ class MoESpec:
     kind: str = "moe"
     identity: int = 0
     correction: Optional[str] = None
-    route_scale: float = 1.0      # with `correction`
+    route_scale: float = 1.0      # with `correction` or scores 'sigmoid'
+    scores: str = "softmax"       # 'softmax' | 'sigmoid'
+    groups: int = 1
+    group_keep: int = 1
     activation: str = "silu"      # of the experts, as SwiGLUSpec's
     limit: float = 0.0
     slope: float = 0.0
@@ -287,8 +297,8 @@ class DiffAttentionSpec:
     """Causal grouped-query differential attention: every head has two query/key maps of `head_dim` entries
     each over the head's one set of values; the head's output is map 1 minus `lam` times map 2 (lam =
     exp(lq1 . lk1) - exp(lq2 . lk2) + diff, one number a layer), divided by its root mean square over
-    `value_dim` and scaled by 1 - diff.  q, k and v have biases; each map of q and k is RMS-normed over
-    head_dim with a weight shared by heads and maps, then rotated."""
+    `value_dim` and scaled by 1 - diff.  q, k and v may have biases; each map of q and k may be RMS-normed over
+    head_dim with a weight shared by heads and maps (q_norm, k_norm), and may then be rotated (position)."""
     hidden_size: int
     num_heads: int
     num_kv_heads: int
@@ -300,8 +310,8 @@ class DiffAttentionSpec:
     q_proj: str                   # [heads * 2 * head_dim, hidden], head by head [map 1 | map 2]; bias: name + ".b"
     k_proj: str
     v_proj: str
-    q_norm: str
-    k_norm: str
+    q_norm: Optional[str]
+    k_norm: Optional[str]
     lam_q1: str
     lam_k1: str
     lam_q2: str
@@ -310,14 +320,18 @@ class DiffAttentionSpec:
     position: Optional[object] = None
     window: int = 0
     kind: str = "diff_attention"
+    bias: bool = True
 
     def tensors(self) -> TensorTable:
         H, G, n, dv, d = self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, self.hidden_size
-        t: TensorTable = {self.q_proj: ((H * 2 * n, d), "matrix"), self.q_proj + ".b": ((H * 2 * n,), "normal:0:0.02"),
-                          self.k_proj: ((G * 2 * n, d), "matrix"), self.k_proj + ".b": ((G * 2 * n,), "normal:0:0.02"),
-                          self.v_proj: ((G * dv, d), "matrix"), self.v_proj + ".b": ((G * dv,), "normal:0:0.02"),
-                          self.q_norm: ((n,), "norm"), self.k_norm: ((n,), "norm"),
-                          self.o_proj: ((d, H * dv), "matrix")}
+        t: TensorTable = {self.o_proj: ((d, H * dv), "matrix")}
+        for name, rows in ((self.q_proj, H * 2 * n), (self.k_proj, G * 2 * n), (self.v_proj, G * dv)):
+            t[name] = ((rows, d), "matrix")
+            if self.bias:
+                t[name + ".b"] = ((rows,), "normal:0:0.02")
+        for name in (self.q_norm, self.k_norm):
+            if name is not None:
+                t[name] = ((n,), "norm")
         for name in (self.lam_q1, self.lam_k1, self.lam_q2, self.lam_k2):
             t[name] = ((n,), "normal:0:0.1")
         if self.position is not None:
@@ -327,17 +341,23 @@ class DiffAttentionSpec:
 
 @dataclass(frozen=True)
 class ActMLPSpec:
-    """Ungated feed-forward: down(act(up x)), no biases; act 'relu2' is the square of relu, 'gelu_tanh' the tanh form of GELU."""
+    """Ungated feed-forward: down(act(up x)); act 'relu2' is the square of relu, 'gelu_tanh' the tanh form of GELU; with `bias` both
+    products have one (name + ".b")."""
     hidden_size: int
     intermediate_size: int
     up_proj: str
     down_proj: str
     activation: str = "relu2"
     kind: str = "act_mlp"
+    bias: bool = False
 
     def tensors(self) -> TensorTable:
-        return {self.up_proj: ((self.intermediate_size, self.hidden_size), "matrix"),
-                self.down_proj: ((self.hidden_size, self.intermediate_size), "matrix")}
+        t: TensorTable = {self.up_proj: ((self.intermediate_size, self.hidden_size), "matrix"),
+                          self.down_proj: ((self.hidden_size, self.intermediate_size), "matrix")}
+        if self.bias:
+            t[self.up_proj + ".b"] = ((self.intermediate_size,), "normal:0:0.02")
+            t[self.down_proj + ".b"] = ((self.hidden_size,), "normal:0:0.02")
+        return t
 
 
 @dataclass(frozen=True)
@@ -732,6 +752,32 @@ class DepthAverageSpec:
 
 
 @dataclass(frozen=True)
+class StreamsSpec:
+    """The residual as `count` streams (hyper-connections), all equal to the embedding's output at the start; the model's output is
+    the norm of their sum.  Every block must be one that reads and writes streams ('hyper')."""
+    count: int
+    hidden_size: int
+    kind: str = "hyper_streams"
+
+    def tensors(self) -> TensorTable:
+        return {}
+
+
+@dataclass(frozen=True)
+class StreamLinkSpec:
+    """How one sublayer is tied to the streams: it reads sum_s read[s] x_s, and its output y goes back as
+    x_t <- sum_s mix[s, t] x_s + m * write[t] * y (m: the layer's residual_mult), all streams at once from the old ones."""
+    count: int
+    read: str                     # [count]
+    write: str                    # [count]
+    mix: str                      # [count, count], from and to
+
+    def tensors(self) -> TensorTable:
+        n = self.count
+        return {self.read: ((n,), f"normal:{1.0 / n}:0.2"), self.write: ((n,), "normal:1:0.2"), self.mix: ((n, n), f"normal:{1.0 / n}:0.2")}
+
+
+@dataclass(frozen=True)
 class LayerSpec:
     """One block: which parts and how they are arranged ('pre_norm': x += mixer(norm(x));
     x += ffn(norm(x)), the reference's order, runtime/src/text_model.cpp:146-168; 'parallel':
@@ -743,7 +789,8 @@ class LayerSpec:
     mixer_gate / ffn_gate name W [width, width], the bias is name + ".b".
     'post_norm': x += mixer_norm(mixer(x)); x += ffn_norm(feed_forward(x)): the parts read the stream itself and the norms
     sit on their outputs.
-    'sandwich_norm': x += mixer_post_norm(mixer(mixer_norm(x))); x += ffn_post_norm(feed_forward(ffn_norm(x)))."""
+    'sandwich_norm': x += mixer_post_norm(mixer(mixer_norm(x))); x += ffn_post_norm(feed_forward(ffn_norm(x))).
+    'hyper': the pre-norm order on several residual streams, each part tied to them by mixer_link / ffn_link (StreamLinkSpec)."""
     mixer: object
     feed_forward: object
     mixer_norm: object
@@ -756,10 +803,13 @@ class LayerSpec:
     ffn_gate: Optional[str] = None
     mixer_post_norm: object = None
     ffn_post_norm: object = None
+    mixer_link: Optional[StreamLinkSpec] = None
+    ffn_link: Optional[StreamLinkSpec] = None
 
     def tensors(self) -> TensorTable:
         t: TensorTable = {}
-        for part in (self.mixer_norm, self.mixer, self.mixer_post_norm, self.ffn_norm, self.feed_forward, self.ffn_post_norm):
+        for part in (self.mixer_norm, self.mixer, self.mixer_post_norm, self.ffn_norm, self.feed_forward, self.ffn_post_norm, self.mixer_link,
+                     self.ffn_link):
             if part is not None:
                 t.update(part.tensors())
         width = getattr(self.mixer_norm, "size", None)
@@ -791,6 +841,7 @@ class ModelSpec:
     loop: Optional[LoopSpec] = None           # where and how the stream re-enters a stretch of layers that runs again
     logit_scale: float = 1.0                  # a fixed factor on the logits
     depth_average: Optional[DepthAverageSpec] = None    # the stream after each run as a weighted sum of the runs' results
+    streams: Optional[StreamsSpec] = None     # the residual as several streams
 
     def __post_init__(self):
         if self.order is None:
