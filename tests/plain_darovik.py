@@ -13,6 +13,7 @@ import math
 import torch
 
 F64 = torch.float64
+CLEAR = 0.025            # how far apart the numbers a router's choice hangs on must lie for the choice to be no close call
 
 
 def unit(x, eps):
@@ -38,10 +39,16 @@ def write_streams(X, mix, out, y, mult):
 # ------------------------------------------------------------------ attention
 
 def softmax_with_sink(scores, sink):
-    """Weights over the keys when the denominator also holds exp(sink); they sum to less than one."""
-    top = torch.maximum(scores.max(), sink)
+    """Weights over the keys (the last dimension) when the denominator also holds exp(sink); they sum to less than one."""
+    top = torch.maximum(scores.amax(dim=-1, keepdim=True), sink)
     e = torch.exp(scores - top)
-    return e / (e.sum() + torch.exp(sink - top))
+    return e / (e.sum(dim=-1, keepdim=True) + torch.exp(sink - top))
+
+
+def sees(T, window):
+    """[T, T]: whether token i sees token j; j <= i, and with a window i - j < window."""
+    d = torch.arange(T)[:, None] - torch.arange(T)[None, :]
+    return (d >= 0) & (d < window) if window else d >= 0
 
 
 def latent_attention(h, W, p, m, eps):
@@ -52,20 +59,15 @@ def latent_attention(h, W, p, m, eps):
     k = (c @ W[p + "uk"].T).reshape(T, H, n)
     v = (c @ W[p + "uv"].T).reshape(T, H, dv)
     out = torch.zeros(T, H, dv, dtype=F64)
-    for i in range(T):
-        for a in range(H):
-            w = softmax_with_sink((k[: i + 1, a] @ q[i, a]) * float(m["scale"]), W[p + "sink"][a])
-            out[i, a] = w @ v[: i + 1, a]
+    for a in range(H):
+        s = (q[:, a] @ k[:, a].T) * float(m["scale"])
+        out[:, a] = softmax_with_sink(s.masked_fill(~sees(T, 0), -math.inf), W[p + "sink"][a]) @ v[:, a]
     return out.reshape(T, H * dv) @ W[p + "o"].T
 
 
 def softmax_window(q, k, v, scale, window):
     """One map: q [T, n], k [T, n], v [T, m]; token i sees j with 0 <= i - j < window (all j <= i when window is 0)."""
-    out = torch.zeros(q.shape[0], v.shape[1], dtype=F64)
-    for i in range(q.shape[0]):
-        lo = max(0, i - window + 1) if window else 0
-        out[i] = torch.softmax((k[lo: i + 1] @ q[i]) * scale, dim=0) @ v[lo: i + 1]
-    return out
+    return torch.softmax(((q @ k.T) * scale).masked_fill(~sees(q.shape[0], window), -math.inf), dim=-1) @ v
 
 
 def difference_factor(W, p, diff):
@@ -127,6 +129,7 @@ def routed_ff(h, W, p, f, clear=None):
     each token's choice is no close call."""
     s_all = torch.sigmoid(h @ W[p + "router"].T)
     out = torch.zeros_like(h)
+    every = torch.stack([gated_expert(h, W, f"{p}e{e}.") for e in range(s_all.shape[1])])
     gaps = []
     for t in range(h.shape[0]):
         idx, gap = choose(s_all[t], W[p + "correction"], f["router"])
@@ -134,9 +137,9 @@ def routed_ff(h, W, p, f, clear=None):
         w = s_all[t][idx]
         w = w / (w.sum() + 1e-20) * float(f["router"]["scale"])
         for e, we in zip(idx.tolist(), w):
-            out[t] += we * gated_expert(h[t: t + 1], W, f"{p}e{e}.")[0]
+            out[t] += we * every[e, t]
     if clear is not None:
-        clear.append(torch.tensor(gaps) > 0.01)
+        clear.append(torch.tensor(gaps) > CLEAR)
     return out
 
 
