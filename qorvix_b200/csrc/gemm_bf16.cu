@@ -39,6 +39,7 @@ struct GemmArgs {
   int bn;                  // persistent kernel: columns of a tile (a multiple of 16, at most its BN)
   int act = 0;             // the fused activation of a gate/up product: 0 SiLU, 1 the tanh form of GELU, 2 clamped (below)
   float limit = 0.f, slope = 0.f;
+  const float* bias = nullptr;   // EPI 2: one number per feature added before the activation `act` (0: square of relu, 1: tanh form of GELU); null: none
 };
 
 // What the fused rotary epilogue of the QKV product needs: C's columns are H query heads, Hkv key
@@ -69,8 +70,9 @@ struct NormArgs {
 
 // Few tokens.  BN: columns of the accumulator (token rows per tile, padded).  The wide operand is
 // the weight matrix (features) and the narrow one the tokens, so the tile is C^T.
-// SWIGLU: the weight rows come in groups of 32 (16 gate rows, then the 16 up rows of the same
+// EPI 1: the weight rows come in groups of 32 (16 gate rows, then the 16 up rows of the same
 // features); the epilogue writes silu(gate) * up, so C has half as many features as W has rows.
+// EPI 2: the epilogue writes act(sum + bias), an ungated activation.  EPI 0: the sums as they are.
 // bfloat16 output: the fast exponential's error (a few float32 ulp) vanishes in the rounding
 __device__ __forceinline__ float silu_mul(float g, float u) { return __fdividef(g, 1.0f + __expf(-g)) * u; }
 // act 0: silu(g) * u; act 1: gelu_tanh(g) * u = 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))) * u;
@@ -85,7 +87,14 @@ __device__ __forceinline__ float glu_mul(float g, float u, int act, float limit,
   return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * g * g, g, g))) * u;
 }
 
-template <int BN, int STAGES, typename TC, bool SWIGLU>
+// An ungated activation of EPI 2: 0 the square of relu, 1 the tanh form of GELU.
+__device__ __forceinline__ float ungated_act(float z, int act) {
+  if (act == 1) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z)));
+  const float v = fmaxf(z, 0.f);
+  return v * v;
+}
+
+template <int BN, int STAGES, typename TC, int EPI>
 __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CUtensorMap map_wide,
                                                       const __grid_constant__ CUtensorMap map_narrow,
                                                       const GemmArgs args, const NormArgs norm) {
@@ -261,7 +270,7 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CU
           uint32_t r[16];
           tmem_ld16(taddr + c0, r);
           tmem_wait_ld();
-          if (SWIGLU) {
+          if (EPI == 1) {
             // lanes 0..15 hold gate rows, lanes 16..31 the up rows of the same features
             const int feat = ((wide0 + q * 32) >> 1) + (lane & 15);
 #pragma unroll
@@ -270,6 +279,13 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CU
               const float other = __shfl_xor_sync(0xffffffffu, mine, 16);
               const int t = narrow0 + c0 + j;
               if (lane < 16 && frow && t < ntok) store_out<TC>(C + (size_t)t * args.ldc + feat, glu_mul(mine, other, args.act, args.limit, args.slope));
+            }
+          } else if (EPI == 2 && frow) {
+            const float b = args.bias ? args.bias[wide_row] : 0.f;
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+              const int t = narrow0 + c0 + j;
+              if (t < ntok) store_out<TC>(C + (size_t)t * args.ldc + wide_row, ungated_act(__uint_as_float(r[j]) + b, args.act));
             }
           } else if (frow) {
 #pragma unroll
@@ -370,6 +386,11 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CU
               if (lane == 0) part_s[(warp & 3) * BN + j0 + j] = sq;
             }
           } else {
+            if (EPI == 2) {
+              const float b = args.bias ? args.bias[wide_row] : 0.f;
+#pragma unroll
+              for (int j = 0; j < 16; ++j) acc[j] = ungated_act(acc[j] + b, args.act);
+            }
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               if (narrow0 + j0 + j < ntok) store_out<TC>(C + (size_t)(narrow0 + j0 + j) * args.ldc + wide_row, acc[j]);
@@ -395,10 +416,10 @@ __global__ void __launch_bounds__(192) gemm_tc_kernel(const __grid_constant__ CU
 
 // One row's 32 accumulator columns from `col` on go to C: as they are (the first `ncols` of them),
 // or, with the fused activation, as the 16 values silu(gate) * up of the features col/2 ...
-template <typename TC, bool SWIGLU>
+template <typename TC, int EPI>
 __device__ __forceinline__ void store_chunk(TC* C, int ldc, int row, int col, int ncols, const uint32_t* r, int act = 0, float limit = 0.f,
                                             float slope = 0.f) {
-  if (SWIGLU) {
+  if (EPI == 1) {
     TC* dst = C + (size_t)row * ldc + (col >> 1);
     float a[16];
 #pragma unroll
@@ -550,7 +571,7 @@ struct Share {                                       // a CTA's work: a run of k
 __device__ float* d_split_ws = nullptr;
 __device__ int* d_split_flags = nullptr;
 
-template <int BN, int STAGES, typename TC, bool SWIGLU, bool ROPE = false, bool SHARED = false>
+template <int BN, int STAGES, typename TC, int EPI, bool ROPE = false, bool SHARED = false>
 __global__ void __launch_bounds__(192) gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_x,
                                                                  const __grid_constant__ CUtensorMap map_w,
                                                                  const GemmArgs args, const RopeArgs rope) {
@@ -794,9 +815,22 @@ __global__ void __launch_bounds__(192) gemm_tc_persistent_kernel(const __grid_co
           for (int c0 = 0; c0 < bn; c0 += 32) {
             uint32_t r[32];
             tmem_ld32(taddr + c0, r);                  // a last chunk of 16 columns reads on into unused ones
+            float bias_of_lane = 0.f;                  // EPI 2: the chunk's biases, one a lane, fetched while the sums arrive
+            if (EPI == 2 && args.bias != nullptr && n0 + c0 + lane < N) bias_of_lane = args.bias[n0 + c0 + lane];
             tmem_wait_ld();
+            if (EPI == 2) {
+              if (args.act == 1) {
+#pragma unroll
+                for (int j = 0; j < 32; ++j)
+                  r[j] = __float_as_uint(ungated_act(__uint_as_float(r[j]) + __shfl_sync(0xffffffffu, bias_of_lane, j), 1));
+              } else {
+#pragma unroll
+                for (int j = 0; j < 32; ++j)
+                  r[j] = __float_as_uint(ungated_act(__uint_as_float(r[j]) + __shfl_sync(0xffffffffu, bias_of_lane, j), 0));
+              }
+            }
             if (row >= M || n0 + c0 >= N) continue;
-            store_chunk<TC, SWIGLU>(C, args.ldc, row, n0 + c0, (N - (n0 + c0)) < (bn - c0) ? (N - (n0 + c0)) : (bn - c0), r, args.act, args.limit, args.slope);
+            store_chunk<TC, EPI>(C, args.ldc, row, n0 + c0, (N - (n0 + c0)) < (bn - c0) ? (N - (n0 + c0)) : (bn - c0), r, args.act, args.limit, args.slope);
           }
         }
       }
@@ -826,18 +860,18 @@ int device_sms() {
   return sms;
 }
 
-template <int BN, int STAGES, typename TC, bool SWIGLU = false>
+template <int BN, int STAGES, typename TC, int EPI = 0>
 int launch(const CUtensorMap& mw, const CUtensorMap& mn, const GemmArgs& args, dim3 grid, cudaStream_t st,
            const NormArgs& norm = NormArgs()) {
   constexpr int smem = STAGES * (BM * BK * 2 + BN * BK * 2) + 1024 + 1024;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<BN, STAGES, TC, SWIGLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<BN, STAGES, TC, EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
   // split-K CTAs of a tile (grid.z of them) are one cluster
-  return qv_launch_cluster(gemm_tc_kernel<BN, STAGES, TC, SWIGLU>, grid, dim3(192), (size_t)smem, st, dim3(1, 1, grid.z), mw, mn, args, norm);
+  return qv_launch_cluster(gemm_tc_kernel<BN, STAGES, TC, EPI>, grid, dim3(192), (size_t)smem, st, dim3(1, 1, grid.z), mw, mn, args, norm);
 }
 
 float* g_split_ws = nullptr;             // see qv_gemm_bf16_set_split_workspace
@@ -855,11 +889,11 @@ bool share_tiles(int total_tiles, int num_kb, int bn) {
   return g_split_ws != nullptr && g_split_ctas >= sms && bn <= 128 && total_tiles * 4 <= sms * 3 && total_tiles * 8 >= sms && num_kb >= 64;
 }
 
-template <int BN, int STAGES, typename TC, bool SWIGLU, bool ROPE, bool SHARED>
+template <int BN, int STAGES, typename TC, int EPI, bool ROPE, bool SHARED>
 int launch_persistent_kernel(const CUtensorMap& mx, const CUtensorMap& mw, const GemmArgs& args, int ctas, cudaStream_t st, const RopeArgs& rope) {
   constexpr int smem = STAGES * (BM * BK * 2 + BN * BK * 2) + 1024 + 256;
   static bool configured = false;
-  auto kernel = gemm_tc_persistent_kernel<BN, STAGES, TC, SWIGLU, ROPE, SHARED>;
+  auto kernel = gemm_tc_persistent_kernel<BN, STAGES, TC, EPI, ROPE, SHARED>;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
@@ -868,15 +902,15 @@ int launch_persistent_kernel(const CUtensorMap& mx, const CUtensorMap& mw, const
   return qv_launch(kernel, dim3(ctas), dim3(192), (size_t)smem, st, mx, mw, args, rope);
 }
 
-template <int BN, int STAGES, typename TC, bool SWIGLU, bool ROPE = false>
+template <int BN, int STAGES, typename TC, int EPI, bool ROPE = false>
 int launch_persistent(const CUtensorMap& mx, const CUtensorMap& mw, const GemmArgs& args, int total_tiles, cudaStream_t st,
                       const RopeArgs& rope = RopeArgs()) {
   const int sms = device_sms();
   // tiles are shared only by products with the plain epilogue (the narrow, long ones are output and down projections)
-  if (!SWIGLU && !ROPE && share_tiles(total_tiles, (args.K + BK - 1) / BK, args.bn)) {
+  if (EPI == 0 && !ROPE && share_tiles(total_tiles, (args.K + BK - 1) / BK, args.bn)) {
     return launch_persistent_kernel<BN, STAGES, TC, false, false, true>(mx, mw, args, sms, st, rope);
   }
-  return launch_persistent_kernel<BN, STAGES, TC, SWIGLU, ROPE, false>(mx, mw, args, total_tiles < sms ? total_tiles : sms, st, rope);
+  return launch_persistent_kernel<BN, STAGES, TC, EPI, ROPE, false>(mx, mw, args, total_tiles < sms ? total_tiles : sms, st, rope);
 }
 
 }  // namespace
@@ -936,10 +970,17 @@ static int swap_splits(int tiles, int total_kb, int epilogue, int force_splits, 
 // the tensor-core path does not take (the caller then uses the CUDA-core kernel):
 // K not a multiple of 8 elements, or operands whose rows do not start on 16-byte boundaries.
 static int gemm_bf16_entry(void* C, const void* A, const void* W, const void* packed, int M, int N, int K, int lda, int ldw, int ldc,
-                           int c_dt, int* err, int force_splits, int epilogue, void* stream, float limit = 0.f, float slope = 0.f) {
+                           int c_dt, int* err, int force_splits, int epilogue, void* stream, float limit = 0.f, float slope = 0.f,
+                           const float* bias = nullptr) {
   // epilogue 0: C[M,N] = A W^T.  epilogue 1: W's rows are 16 gate rows / 16 up rows interleaved and
   // C[M,N/2] = silu(gate) * up (bfloat16 out, N a multiple of 32).  epilogue 2: as 1 with the tanh form of GELU, 3: clamped (limit, slope).
-  const int act = epilogue >= 2 ? epilogue - 1 : 0;
+  // epilogue 8, 9: C[M,N] = act(A W^T + bias), bfloat16 out, act the square of relu or the tanh form of GELU (bias may be null).
+  const bool ungated = epilogue == 8 || epilogue == 9;
+  const int act = ungated ? epilogue - 8 : (epilogue >= 2 ? epilogue - 1 : 0);
+  if (ungated) {
+    if (c_dt != QV_DT_BF16) return QV_ERR_UNSUPPORTED;
+    epilogue = 0;
+  }
   if (epilogue == 2 || epilogue == 3) epilogue = 1;
   if (M <= 0 || N <= 0) return 0;
   if (epilogue != 0 && (epilogue != 1 || c_dt != QV_DT_BF16 || (N & 31))) return QV_ERR_UNSUPPORTED;
@@ -948,7 +989,7 @@ static int gemm_bf16_entry(void* C, const void* A, const void* W, const void* pa
   if (c_dt != QV_DT_BF16 && c_dt != QV_DT_F32) return QV_ERR_UNSUPPORTED;
   cudaStream_t st = (cudaStream_t)stream;
   GemmArgs args;
-  args.C = C; args.err = err; args.packed = nullptr; args.bn = 0; args.act = act; args.limit = limit; args.slope = slope;
+  args.C = C; args.err = err; args.packed = nullptr; args.bn = 0; args.act = act; args.limit = limit; args.slope = slope; args.bias = bias;
   args.K = K; args.ldc = ldc;
   const int total_kb = (K + BK - 1) / BK;
   CUtensorMap mw, mn;
@@ -971,6 +1012,11 @@ static int gemm_bf16_entry(void* C, const void* A, const void* W, const void* pa
       return launch<64, 4, bf16, true>(mw, mn, args, grid, st);
     }
     const bool one_wave = tiles * splits <= device_sms();     // every CTA resident at once, one per SM: deeper rings
+    if (ungated) {
+      if (bn == 16) return one_wave ? launch<16, 12, bf16, 2>(mw, mn, args, grid, st) : launch<16, 6, bf16, 2>(mw, mn, args, grid, st);
+      if (bn == 32) return one_wave ? launch<32, 10, bf16, 2>(mw, mn, args, grid, st) : launch<32, 5, bf16, 2>(mw, mn, args, grid, st);
+      return one_wave ? launch<64, 8, bf16, 2>(mw, mn, args, grid, st) : launch<64, 4, bf16, 2>(mw, mn, args, grid, st);
+    }
     if (bn == 16) return one_wave ? SWAP_LAUNCH(16, 12) : SWAP_LAUNCH(16, 6);
     if (bn == 32) return one_wave ? SWAP_LAUNCH(32, 10) : SWAP_LAUNCH(32, 5);
     return one_wave ? SWAP_LAUNCH(64, 8) : SWAP_LAUNCH(64, 4);
@@ -989,6 +1035,7 @@ static int gemm_bf16_entry(void* C, const void* A, const void* W, const void* pa
   if (packed) mn = mw;
   else if (!make_map(&mn, W, N, K, ldw, bn)) return QV_ERR_UNSUPPORTED;
   const int total_tiles = ((M + BM - 1) / BM) * ((N + bn - 1) / bn);
+  if (ungated) return launch_persistent<256, 4, bf16, 2>(mw, mn, args, total_tiles, st);
   if (epilogue == 1) return launch_persistent<256, 4, bf16, true>(mw, mn, args, total_tiles, st);
   if (c_dt == QV_DT_BF16) return launch_persistent<256, 4, bf16, false>(mw, mn, args, total_tiles, st);
   return launch_persistent<256, 4, float, false>(mw, mn, args, total_tiles, st);
@@ -1099,6 +1146,14 @@ extern "C" int qv_gemm_bf16_glu(void* C, const void* A, const void* W, const voi
                                 int* err, int act, float limit, float slope, void* stream) {
   if ((!W && !packed) || act < 0 || act > 2) return QV_ERR_UNSUPPORTED;
   return gemm_bf16_entry(C, A, W, packed, M, N, K, lda, packed ? K : ldw, ldc, QV_DT_BF16, err, 0, act + 1, stream, limit, slope);
+}
+
+// A product with an ungated activation in its epilogue: C [M, N] bfloat16 = act(A W^T + bias), act 0 the square of relu, 1 the tanh
+// form of GELU, bias float32 [N] or null; W as rows (row stride ldw) or packed.
+extern "C" int qv_gemm_bf16_act(void* C, const void* A, const void* W, const void* packed, int M, int N, int K, int lda, int ldw, int ldc,
+                                int* err, int act, const float* bias, void* stream) {
+  if ((!W && !packed) || act < 0 || act > 1) return QV_ERR_UNSUPPORTED;
+  return gemm_bf16_entry(C, A, W, packed, M, N, K, lda, packed ? K : ldw, ldc, QV_DT_BF16, err, 0, 8 + act, stream, 0.f, 0.f, bias);
 }
 
 // ---------------------------------------------------------------- packed weights

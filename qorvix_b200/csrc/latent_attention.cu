@@ -72,12 +72,64 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(
   }
 }
 
+// The same without a rotated part (dr = 0): a warp per token, the latent read four entries at a time where it lies on the vectors'
+// boundaries; up to 1,024 entries stay in registers between the sum and the write.
+template <typename T>
+__global__ void __launch_bounds__(128) latent_rows_kernel(const T* __restrict__ lat0, int ld, T* __restrict__ cache, const float* __restrict__ norm_w,
+                                                          float eps, const int* __restrict__ tok_pos, const int* __restrict__ tok_seg,
+                                                          const int* __restrict__ block_table, int max_blocks, int T_all, int rank, int page) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= T_all) return;
+  const T* lat = lat0 + (size_t)t * ld;
+  const int pos = tok_pos[t];
+  const int pg = block_table[(size_t)tok_seg[t] * max_blocks + pos / page];
+  T* dst = cache + ((size_t)pg * page + (size_t)(pos % page)) * rank;
+  float ss = 0.f;
+  constexpr int MAXV = 8;
+  if (rank % 4 == 0 && rank <= MAXV * 128 && (((uintptr_t)lat | (uintptr_t)dst) & (4 * sizeof(T) - 1)) == 0 && (((uintptr_t)norm_w) & 15) == 0) {
+    float4 v[MAXV];
+#pragma unroll
+    for (int k = 0; k < MAXV; ++k) {
+      const int i = 4 * (lane + 32 * k);
+      v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < rank) {
+        __align__(16) T e[4];
+        if (sizeof(T) == 2) *(uint2*)e = *(const uint2*)(lat + i);
+        else *(uint4*)e = *(const uint4*)(lat + i);
+        v[k] = make_float4(to_f(e[0]), to_f(e[1]), to_f(e[2]), to_f(e[3]));
+      }
+      ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    }
+    const float sc = 1.0f / sqrtf(warp_sum(ss) / (float)rank + eps);
+#pragma unroll
+    for (int k = 0; k < MAXV; ++k) {
+      const int i = 4 * (lane + 32 * k);
+      if (i < rank) {
+        const float4 w = *(const float4*)(norm_w + i);
+        __align__(16) T e[4] = {from_f<T>(v[k].x * sc * w.x), from_f<T>(v[k].y * sc * w.y), from_f<T>(v[k].z * sc * w.z), from_f<T>(v[k].w * sc * w.w)};
+        if (sizeof(T) == 2) *(uint2*)(dst + i) = *(const uint2*)e;
+        else *(uint4*)(dst + i) = *(const uint4*)e;
+      }
+    }
+  } else {
+    for (int i = lane; i < rank; i += 32) { const float v = to_f(lat[i]); ss += v * v; }
+    const float sc = 1.0f / sqrtf(warp_sum(ss) / (float)rank + eps);
+    for (int i = lane; i < rank; i += 32) dst[i] = from_f<T>(to_f(lat[i]) * sc * norm_w[i]);
+  }
+}
+
 extern "C" int qv_latent_prepare(void* proj, int ld, void* q, int ld_q, int kv_off, void* cache, const float* norm_w, float eps,
                                  const float* cos_sin, int table_rows, const int* tok_pos, const int* tok_seg,
                                  const int* block_table, int max_blocks, int T, int H, int dn, int dr, int rank, int rot,
                                  int page, int split_half, int dt, void* stream) {
   if (T <= 0) return 0;
   if (rot < 0 || rot > dr || (rot & 1) || rank <= 0) return QV_ERR_UNSUPPORTED;
+  if (dr == 0)
+    QV_DISPATCH_DT(dt, TT,
+                   return qv_launch(latent_rows_kernel<TT>, dim3((T + 3) / 4), dim3(128), 0, (cudaStream_t)stream, (const TT*)proj + kv_off, ld, (TT*)cache,
+                                    norm_w, eps, tok_pos, tok_seg, block_table, max_blocks, T, rank, page));
   QV_DISPATCH_DT(dt, TT,
                  return qv_launch(latent_prepare_kernel<TT>, dim3(T), dim3(256), 0, (cudaStream_t)stream, (TT*)proj, ld, (TT*)q, ld_q,
                                   kv_off, (TT*)cache, norm_w, eps, (const float2*)cos_sin, table_rows, tok_pos, tok_seg, block_table,

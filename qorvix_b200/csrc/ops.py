@@ -89,6 +89,7 @@ _ARGTYPES = {
     "qv_embed_pos": [_V, _V, _V, _V, _V, _I, _I, _I, _I, _F, _V, _V, _F, _I, _V],
     "qv_glu_act": [_V, _V, _I, _I, _I, _F, _F, _I, _I, _V],
     "qv_gemm_bf16_glu": [_V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _V, _I, _F, _F, _V],
+    "qv_gemm_bf16_act": [_V, _V, _V, _V, _I, _I, _I, _I, _I, _I, _V, _I, _V, _V],
     "qv_sigmoid_gate": [_V, _V, _I, _V, _I, _V, _I, _I, _I, _V],
     "qv_depth_mix": [_V, _V, _V, _L, _V, _I, _V],
     "qv_scale": [_V, _L, _F, _V],
@@ -1498,6 +1499,25 @@ def gemm_bf16_glu(out, x, w_interleaved, packed, n: int, act: int, limit: float,
         return False
     _check(rc, "gemm_bf16_glu")
     return True
+
+
+def gemm_act(out, x, w, packed, n: int, act: int, bias=None) -> None:
+    """out[M, n] = act(x W^T + bias) with an ungated activation (ACT_RELU2 or ACT_GELU_TANH; bias float32 [n] or None): in the product's
+    epilogue on the tensor cores (bfloat16, w as rows or packed), else the product and the activation's pass."""
+    _need_cuda(out, x, w, packed, bias)
+    M, K = x.shape
+    n = n or w.shape[0]
+    assert tuple(out.shape) == (M, n) and x.stride(1) == 1 and out.stride(1) == 1
+    assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == n)
+    if x.dtype == out.dtype == torch.bfloat16 and (packed is not None or w.dtype == torch.bfloat16):
+        rc = _lib("gemm_bf16").qv_gemm_bf16_act(_ptr(out), _ptr(x), _ptr(w) if packed is None else None, _ptr(packed), M, n, K, x.stride(0),
+                                                w.stride(0) if w is not None else K, out.stride(0), _ptr(_gemm_buffers(x.device)["err"]), act,
+                                                _ptr(bias), _stream())
+        if rc != -2:
+            _check(rc, "gemm_act")
+            return
+    gemm(out, x, w, packed, n)
+    activation(out, out, act, bias=bias)
 
 
 def gemm_swiglu(out, x, w_interleaved, packed=None, n: int = 0, act: int = 0, limit: float = 0.0, slope: float = 0.0) -> None:

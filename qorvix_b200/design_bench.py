@@ -1,9 +1,9 @@
-"""Prefill and decode throughput of a Deganex, a Lotirax, a Tubazen, a Lugizen or a Nedasun model at layer sizes that resemble real models, beside the
+"""Prefill and decode throughput of a Deganex, a Lotirax, a Tubazen, a Lugizen, a Nedasun or a Darovik model at layer sizes that resemble real models, beside the
 Llama decoder at equal width, depth and (active) feed-forward size, and the design's kernels alone with their roofline
 fractions beside the Llama kernels they correspond to.
 
-    python bench.py --design deganex|lotirax|tubazen|lugizen|nedasun [--layers-per-kind 2] [--batch 8] [--ctx 1024] [--prefill-tokens 2048]
-    python -m qorvix_b200.design_bench [--design lotirax|tubazen|lugizen|nedasun]
+    python bench.py --design deganex|lotirax|tubazen|lugizen|nedasun|darovik [--layers-per-kind 2] [--batch 8] [--ctx 1024] [--prefill-tokens 2048]
+    python -m qorvix_b200.design_bench [--design lotirax|tubazen|lugizen|nedasun|darovik]
 
 Random bfloat16 weights; timing with CUDA events after warm-up; kernels alone are timed in captured chains over
 buffers larger than L2 (kernel_bench.timed_chain).  Figures go out as one JSON line.
@@ -116,10 +116,13 @@ def _ctx(seg_lens, pos0, device="cuda"):
         tok_pos=torch.cat([torch.arange(p, p + n, **i32) for p, n in zip(pos0, seg_lens)]))
 
 
-def latent_attention_case(seg_lens, ctx_len, peaks, page=16, window=0, gated=True) -> dict:
+def latent_attention_case(seg_lens, ctx_len, peaks, page=16, window=0, gated=True, sinks=False) -> dict:
     """Latent attention of the given segments, each ending at ctx_len cached tokens (prepare excluded); window > 0: the last
-    `window` keys only; gated False: without the output gate."""
+    `window` keys only; gated False: without the output gate; sinks: without the rotated part, with a sink per head and softmax
+    weights of 24 bits."""
     H, dn, dr, dv, rank = ATTN["heads"], ATTN["dim"], ATTN["rot_dim"], ATTN["vdim"], ATTN["kv_rank"]
+    dr = 0 if sinks else dr
+    more = dict(sink=torch.randn(H, device="cuda"), weight_terms=3) if sinks else {}
     S, T = len(seg_lens), sum(seg_lens)
     blocks = -(-ctx_len // page)
     row_bytes = (rank + dr) * 2
@@ -136,7 +139,7 @@ def latent_attention_case(seg_lens, ctx_len, peaks, page=16, window=0, gated=Tru
     wuk_t = wuk.view(H, dn, rank).transpose(1, 2).contiguous()
     out = torch.empty(T, H * dv, device="cuda", dtype=torch.bfloat16)
     us = kb.timed_chain(lambda i: ops.latent_attention(out, q, gate, caches[i % copies], wuk, wuv, ctx, table, H, dn, dr, dv, rank, page, window,
-                                                       ATTN["scale"], wuk_t=wuk_t), launches=8)
+                                                       ATTN["scale"], wuk_t=wuk_t, **more), launches=8)
     seen = lambda pos: min(pos + 1, window) if window else pos + 1                      # keys a query at `pos` sees
     pairs = sum(seen(ctx_len - n + i) for n in seg_lens for i in range(n))              # (query, key) pairs per head
     flops = H * pairs * (2.0 * (rank + dr) + 2.0 * rank) + T * H * 2.0 * rank * (dn + dv)
@@ -168,9 +171,10 @@ def scan_case(kind, seg_lens, peaks) -> dict:
     return kb._figures(us, nbytes, 4.0 * T * H * dk * dv, peaks)
 
 
-def experts_case(T, peaks, identity=0) -> dict:
+def experts_case(T, peaks, identity=0, groups=None) -> dict:
     """Both products of the routed experts for T tokens (router and grouping included, shared expert excluded); identity > 0: the
-    router that scores all experts, with that many identity experts (whose choices take no product) and clamped activations."""
+    router that scores all experts, with that many identity experts (whose choices take no product) and clamped activations;
+    groups (count, keep): the router of corrected sigmoids that chooses within the best groups."""
     E, top, ff, d = MOE["router"]["experts"], MOE["router"]["top"], MOE["expert"]["ff"], WIDTH
     wbytes = E * 3 * ff * d * 2
     copies = max(2, int(2.5 * kb.L2_BYTES // wbytes) + 1)
@@ -189,10 +193,14 @@ def experts_case(T, peaks, identity=0) -> dict:
     y = torch.empty(R, d, device="cuda", dtype=torch.float32)
     delta = torch.empty(T, d, device="cuda", dtype=torch.float32)
     corr = torch.zeros(E + identity, device="cuda") if identity else None
+    route = {}
+    if groups:
+        corr, route = torch.randn(E, device="cuda") * 0.1, dict(sigmoid=True, groups=groups[0], keep=groups[1])
+        router.mul_(d ** -0.5)
     glu = dict(act=ops.GLU_CLAMPED, limit=7.0, slope=1.702) if identity else {}
 
     def run(i):
-        ops.moe_route(top_idx, top_w, None, x, router, None, correction=corr, w_scale=2.5)
+        ops.moe_route(top_idx, top_w, None, x, router, None, correction=corr, w_scale=2.5, **route)
         ops.moe_group(row_token, slot_row, tiles, top_idx, scratch, E, tile_rows)
         ops.moe_experts_tc(True, act, x, wg[i % copies], wu[i % copies], row_token, tiles, **glu)
         ops.moe_experts_tc(False, y, act, wd[i % copies], None, row_token, tiles)
@@ -833,6 +841,135 @@ def run_nedasun(args, peaks) -> dict:
     return res
 
 
+# ------------------------------------------------------------------ Darovik
+# Latent attention of 16 heads of 128 over a latent of 512 without positions and with sinks; differential attention of 16 heads of
+# two 64-wide maps over 128 values on four key/value heads with a window of 1,024; an ungated feed-forward of 12,288 with biases, or 64
+# gated experts of 1,408 in eight groups of which four are open and 6 experts serve a token; two residual streams; the two middle
+# layers run twice.
+DAR_LATENT = {"heads": 16, "dim": 128, "vdim": 128, "kv_rank": 512, "scale": 128 ** -0.5}
+DAR_ATTN = {k: v for k, v in LOT_ATTN.items() if k != "rot"}
+DAR_DENSE = {"kind": "dense", "ff": 12288}
+DAR_MOE = {"kind": "moe", "expert": {"ff": 1408}, "router": {"experts": 64, "groups": {"count": 8, "keep": 4}, "scale": 2.5, "top": 6}}
+DAR_STREAMS = 2
+
+
+def darovik_config() -> dict:
+    layers = [{"type": "latent_attention", "mixer": DAR_LATENT, "mlp": DAR_DENSE}, {"type": "attention", "mixer": DAR_ATTN, "mlp": DAR_MOE}] * 2
+    return {"architecture": "Darovik", "vocab": VOCAB, "width": WIDTH, "norm": {"eps": 1e-5}, "residual_mult": 0.25, "streams": DAR_STREAMS,
+            "layers": layers, "loop": {"start": 1, "stop": 3, "times": 2}}
+
+
+def darovik_lotirax_config() -> dict:
+    """The closest model's layers in the same order with feed-forwards of the same number of weights (its dense one has a gate, its
+    experts have none)."""
+    dense, moe = {"kind": "dense", "ff": 8192}, {"kind": "moe", "expert": {"ff": 2112}, "router": {"experts": 64, "top": 6}}
+    layers = [{"type": "attention", "mixer": LOT_ATTN, "mlp": f} for f in (dense, moe, dense, moe)]
+    return dict(lotirax_config(), layers=layers)
+
+
+def cache_rows_case(T, peaks, page=16) -> dict:
+    """Keys and values of T tokens of one request from the projection's columns into the pages."""
+    a = DAR_ATTN
+    H, G, n, dv = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+    cols, width = (H + G) * 2 * n + G * dv, G * (2 * n + dv)
+    copies = max(2, min(8, int(2.5 * kb.L2_BYTES // (T * width * 4)) + 1))
+    projs = torch.randn(copies, T, cols, device="cuda", dtype=torch.bfloat16)
+    blocks = -(-T // page)
+    caches = torch.zeros(copies, blocks + 1, page, width, device="cuda", dtype=torch.bfloat16)
+    table = torch.arange(blocks, dtype=torch.int32, device="cuda").view(1, blocks)
+    ctx = _ctx([T], [0])
+    us = kb.timed_chain(lambda i: ops.cache_rows(caches[i % copies], projs[i % copies][:, H * 2 * n:], ctx, table, page), launches=8)
+    return kb._figures(us, T * width * 4, 0.0, peaks)
+
+
+def latent_prepare_case(T, peaks, page=16, rotated=False) -> dict:
+    """The latents' norm and cache write of T tokens of one request; rotated: with the shared key part and the heads' query parts."""
+    H, dn, rank = ATTN["heads"], ATTN["dim"], ATTN["kv_rank"]
+    dr = ATTN["rot_dim"] if rotated else 0
+    cols = H * (dn + dr) + rank + dr
+    copies = max(2, min(8, int(2.5 * kb.L2_BYTES // (T * (rank + dr) * 4)) + 1))
+    projs = torch.randn(copies, T, cols, device="cuda", dtype=torch.bfloat16)
+    blocks = -(-T // page)
+    caches = torch.zeros(copies, blocks + 1, page, rank + dr, device="cuda", dtype=torch.bfloat16)
+    table = torch.arange(blocks, dtype=torch.int32, device="cuda").view(1, blocks)
+    ctx = _ctx([T], [0])
+    cos_sin = torch.ones(T, dr // 2, 2, device="cuda") if rotated else None
+    w = torch.ones(rank, device="cuda")
+    us = kb.timed_chain(lambda i: ops.latent_prepare(projs[i % copies], projs[i % copies][:, : H * (dn + dr)], H * (dn + dr), caches[i % copies], w, 1e-5,
+                                                     cos_sin, ctx, table, H, dn, dr, rank, dr, page), launches=8)
+    return kb._figures(us, T * ((rank + dr) * 4 + H * dr * 4), 0.0, peaks)
+
+
+def stream_pass_case(T, peaks, streams=DAR_STREAMS) -> dict:
+    """A sublayer's output back to all streams, which are mixed, and the next sublayer's normed input, in one pass."""
+    d, S = WIDTH, streams
+    copies = max(2, min(8, int(2.5 * kb.L2_BYTES // (T * d * (8 * S + 4))) + 1))
+    res = torch.randn(copies, T, S, d, device="cuda", dtype=torch.float32)
+    y = torch.randn(copies, T, d, device="cuda", dtype=torch.bfloat16)
+    h = torch.empty(copies, T, d, device="cuda", dtype=torch.bfloat16)
+    w, read = torch.ones(d, device="cuda"), torch.full((S,), 1.0 / S, device="cuda")
+    write = torch.cat([torch.eye(S).reshape(-1), torch.full((S,), 1e-3)]).cuda()
+    us = kb.timed_chain(lambda i: ops.stream_pass(h[i % copies], res[i % copies], read, weight=w, eps=1e-5, y=y[i % copies], write_coef=write), launches=8)
+    return kb._figures(us, T * d * (8 * S + 4), 0.0, peaks)
+
+
+def biased_up_case(T, peaks, bias=True, fused=True) -> dict:
+    """The ungated feed-forward's first product and its activation, with the bias or without, in one kernel or (fused False) in two."""
+    ff, d = DAR_DENSE["ff"], WIDTH
+    copies = max(2, int(2.5 * kb.L2_BYTES // (ff * d * 2)) + 1)
+    ws = [ops.pack_weight(torch.randn(ff, d, device="cuda", dtype=torch.bfloat16) * 0.02) for _ in range(copies)]
+    x = torch.randn(T, d, device="cuda", dtype=torch.bfloat16)
+    b = torch.randn(ff, device="cuda") if bias else None
+    out = torch.empty(T, ff, device="cuda", dtype=torch.bfloat16)
+
+    def run(i):
+        if fused:
+            ops.gemm_act(out, x, None, ws[i % copies], ff, ops.ACT_RELU2, b)
+        else:
+            ops.gemm(out, x, None, ws[i % copies], ff)
+            ops.activation(out, out, ops.ACT_RELU2, bias=b)
+    us = kb.timed_chain(run, launches=8)
+    return kb._figures(us, ff * d * 2 + T * (d + ff) * 2, 2.0 * T * ff * d, peaks)
+
+
+def run_darovik(args, peaks) -> dict:
+    n_runs = 6
+    sizes = (args.batch, args.ctx, args.prefill_tokens, args.steps, args.warmup)
+    T, B, C = args.prefill_tokens, args.batch, args.ctx
+    res = {"darovik": model_throughput(darovik_config(), *sizes), "lotirax_equal_size": model_throughput(darovik_lotirax_config(), *sizes),
+           "llama_equal_size": model_throughput(lotirax_llama_config(n_runs), *sizes)}
+    groups = (DAR_MOE["router"]["groups"]["count"], DAR_MOE["router"]["groups"]["keep"])
+    many = {f"latent_prefill_t{T}": lambda **k: latent_attention_case([T], T, peaks, gated=False, **k),
+            f"latent_prefill_t{T // 4}_ctx{T}": lambda **k: latent_attention_case([T // 4], T, peaks, gated=False, **k),
+            f"latent_decode_b{B}_ctx{C}": lambda **k: latent_attention_case([1] * B, C, peaks, gated=False, **k),
+            f"latent_decode_b{8 * B}_ctx{C}": lambda **k: latent_attention_case([1] * (8 * B), C, peaks, gated=False, **k)}
+    res["kernels"] = {n: f(sinks=True) for n, f in many.items()}
+    res["kernels"].update({
+        f"diff_attention_prefill_t{T}": diff_attention_case([T], T, peaks), f"diff_attention_decode_b{B}_ctx{C}": diff_attention_case([1] * B, C, peaks),
+        f"latent_prepare_t{T}": latent_prepare_case(T, peaks), f"latent_prepare_t{B}": latent_prepare_case(B, peaks),
+        f"cache_rows_t{T}": cache_rows_case(T, peaks), f"cache_rows_t{B}": cache_rows_case(B, peaks),
+        f"stream_pass_t{T}": stream_pass_case(T, peaks), f"stream_pass_t{B}": stream_pass_case(B, peaks),
+        f"stream_pass_4_streams_t{T}": stream_pass_case(T, peaks, 4), f"stream_pass_4_streams_t{B}": stream_pass_case(B, peaks, 4),
+        f"experts_prefill_t{T}": experts_case(T, peaks, groups=groups), f"experts_decode_b{B}": experts_case(B, peaks, groups=groups),
+        f"biased_up_t{T}": biased_up_case(T, peaks), f"biased_up_t{B}": biased_up_case(B, peaks),
+    })
+    # the like kernels of the closest designs at the same sizes: Deganex's latent attention (rotated part, no sinks, rounded weights) and
+    # experts, Lotirax's preparing kernel and ungated product, the pre-norm decoders' norm pass
+    res["like_kernels"] = {n: f() for n, f in many.items()}
+    res["like_kernels"].update({
+        f"latent_prepare_t{T}": latent_prepare_case(T, peaks, rotated=True), f"latent_prepare_t{B}": latent_prepare_case(B, peaks, rotated=True),
+        f"diff_prepare_t{T}": diff_prepare_case(T, peaks), f"diff_prepare_t{B}": diff_prepare_case(B, peaks),
+        f"add_rmsnorm_t{T}": add_rmsnorm_case(T, peaks), f"add_rmsnorm_t{B}": add_rmsnorm_case(B, peaks),
+        f"experts_prefill_t{T}": experts_case(T, peaks), f"experts_decode_b{B}": experts_case(B, peaks),
+        f"ungated_up_t{T}": biased_up_case(T, peaks, False, False), f"ungated_up_t{B}": biased_up_case(B, peaks, False, False),
+    })
+    from .config import LlamaConfig
+    like = kb.headline_kernels(LlamaConfig.from_dict(lotirax_llama_config(n_runs)), B, C, T, peaks)
+    ops.check_kernel_errors()
+    res["llama_kernels"] = {k: v for k, v in like.items() if "attention" in k or "gate_up" in k or "down" in k}
+    return res
+
+
 def run(args, peaks) -> dict:
     n_layers = 3 * args.layers_per_kind
     res = {"deganex": model_throughput(deganex_config(args.layers_per_kind), args.batch, args.ctx, args.prefill_tokens, args.steps, args.warmup),
@@ -856,7 +993,7 @@ def run(args, peaks) -> dict:
 def main(argv=None, peaks=None, extra=None) -> int:
     """extra: a callable whose dict (the clocks sampled during the run, for instance) joins the JSON line."""
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("--design", default="deganex", choices=["deganex", "lotirax", "tubazen", "lugizen", "nedasun"])
+    ap.add_argument("--design", default="deganex", choices=["deganex", "lotirax", "tubazen", "lugizen", "nedasun", "darovik"])
     ap.add_argument("--layers-per-kind", type=int, default=2)
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--ctx", type=int, default=1024)
@@ -873,6 +1010,8 @@ def main(argv=None, peaks=None, extra=None) -> int:
         res, model = run_lugizen(args, peaks), f"Lugizen, width {WIDTH}, {3 * args.layers_per_kind} layers"
     elif args.design == "nedasun":
         res, model = run_nedasun(args, peaks), f"Nedasun, width {WIDTH}, {2 * args.layers_per_kind} layers"
+    elif args.design == "darovik":
+        res, model = run_darovik(args, peaks), f"Darovik, width {WIDTH}, 4 layers of which 2 run twice, {DAR_STREAMS} streams"
     else:
         res, model = run(args, peaks), f"Deganex, width {WIDTH}, {3 * args.layers_per_kind} layers"
     d = res[args.design]

@@ -67,8 +67,8 @@ class SwiGLU(FeedForward):
 
 
 class ActMLP(FeedForward):
-    """Ungated feed-forward: down(act(up x)), the activation (the square of relu, or the tanh form of GELU) as a pass of
-    its own, which also adds the up product's bias where there is one; the down product's bias is offered to the block."""
+    """Ungated feed-forward: down(act(up x)), the up product's bias, where there is one, and the activation (the square of
+    relu, or the tanh form of GELU) in that product's epilogue where the kernel takes it, else a pass of their own; the down product's bias is offered to the block."""
 
     def __init__(self, spec, source, rt):
         acts = {"relu2": ops.ACT_RELU2, "gelu_tanh": ops.ACT_GELU_TANH}
@@ -83,8 +83,8 @@ class ActMLP(FeedForward):
         self.output_bias = source.get(spec.down_proj + ".b", dtype=torch.float32) if bias else None
 
     def forward(self, x, ctx, with_bias: bool = True):
-        act = self.up(x, out_dtype=self.rt.dtype)
-        ops.activation(act, act, self.act, bias=self.up_bias)
+        act = torch.empty((x.shape[0], self.up.out_features), device=x.device, dtype=self.rt.dtype)
+        ops.gemm_act(act, x, self.up.weight, self.up.packed, self.up.out_features, self.act, self.up_bias)
         if self.output_bias is None or not with_bias:
             return self.down(act, out_dtype=self.rt.dtype)
         y = self.down(act, out_dtype=torch.float32)

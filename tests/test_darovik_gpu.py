@@ -209,6 +209,25 @@ def test_activation_with_and_without_a_bias(cols, kind, dtype):
         close(buf.float(), want, dtype, "activation")
 
 
+@pytest.mark.parametrize("kind", [ops.ACT_RELU2, ops.ACT_GELU_TANH])
+@pytest.mark.parametrize("M,N,K", [(1, 88, 72), (8, 512, 2048), (17, 130, 264), (40, 1000, 72), (64, 4096, 512), (65, 88, 72), (200, 1000, 264), (300, 512, 1024), (129, 37, 64), (5, 40, 70)])
+@pytest.mark.parametrize("packed", [True, False])
+def test_product_with_an_ungated_activation_in_its_epilogue(M, N, K, packed, kind):
+    """Few tokens with and without splits along K, many tokens in whole and ragged tiles, rows and packed tiles, a bias or none; and a
+    size the tensor-core kernel refuses (K no multiple of 8), which takes two kernels."""
+    x, w, b = bf(rnd(M, K, seed=M)), bf(rnd(N, K, seed=N) * K ** -0.5), rnd(N, seed=K)
+    if packed and K % 8:
+        pytest.skip("no packed tiles for this size")
+    on = lambda t: t.to(torch.bfloat16).to(DEV)
+    for bias in (b, None):
+        z = x.double() @ w.double().T + (bias.double() if bias is not None else 0.0)
+        want = z.clamp(min=0) ** 2 if kind == ops.ACT_RELU2 else torch.nn.functional.gelu(z, approximate="tanh")
+        out = torch.full((M, N), float("nan"), dtype=torch.bfloat16, device=DEV)
+        ops.gemm_act(out, on(x), None if packed else on(w), ops.pack_weight(on(w)) if packed else None, N, kind, bias.to(DEV) if bias is not None else None)
+        ops.check_kernel_errors()
+        close(out.float(), want, torch.bfloat16, "product", loose=0.3)
+
+
 MOE_CASES = [(dh.moe(), 37), (dh.moe(experts=1, top=1, ff=30, groups=(1, 1)), 5), (dh.moe(experts=8, top=3, ff=16, groups=(4, 2)), 1),
              (dh.moe(experts=16, top=4, ff=64, groups=(4, 1)), 300), (dh.moe(experts=7, top=2, ff=13, groups=None), 70),
              (dh.moe(experts=12, top=5, ff=24, groups=(12, 5), scale=1.0), 40), (dh.moe(experts=72, top=6, ff=8, groups=(36, 7)), 50)]
