@@ -591,30 +591,58 @@ __global__ void __launch_bounds__(LT_WARPS * 32) latent_attention_tc_kernel(
 
 // lat[row][:] (bfloat16) = the partial results of a (token, head) row merged: sum_s e^(m_s - M) o_s / (sum_s e^(m_s - M) l_s +
 // e^(sink[head] - M) where there are sinks)
+// The slices' factors are worked out once by all threads, then every thread reads its columns of four slices at a time.
 __global__ void __launch_bounds__(128) latent_merge_kernel(bf16* __restrict__ lat, const float* __restrict__ part_o,
                                                            const float* __restrict__ part_ml, int rank, int splits, int total_rows,
                                                            const float* __restrict__ sink, int H) {
+  extern __shared__ float merge_w[];                       // one factor per slice
+  __shared__ float red[8];
   pdl_wait();
   pdl_launch_dependents();
   const size_t row = blockIdx.x;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const float sk = sink ? sink[row % H] : -INFINITY;
-  float M = sk;
-  for (int s = 0; s < splits; ++s) M = fmaxf(M, part_ml[2 * ((size_t)s * total_rows + row)]);
-  float L = sink ? expf(sk - M) : 0.f;
-  for (int s = 0; s < splits; ++s) {
-    const float m = part_ml[2 * ((size_t)s * total_rows + row)];
-    if (m != -INFINITY) L += expf(m - M) * part_ml[2 * ((size_t)s * total_rows + row) + 1];
+  if (splits == 1) {                                       // nothing to merge: divide (and take the sink in)
+    const float2 ml = *(const float2*)(part_ml + 2 * row);
+    const float top = fmaxf(ml.x, sk), w = expf(ml.x - top);
+    const float f = w / (w * ml.y + (sink ? expf(sk - top) : 0.f));
+    for (int r = tid * 2; r < rank; r += 256) {
+      const float2 v = *(const float2*)(part_o + row * rank + r);
+      *(__nv_bfloat162*)(lat + row * rank + r) = __floats2bfloat162_rn(v.x * f, v.y * f);
+    }
+    return;
   }
-  const float inv = 1.0f / L;
-  for (int r = threadIdx.x * 2; r < rank; r += blockDim.x * 2) {
+  float M = sk;
+  for (int s = tid; s < splits; s += 128) M = fmaxf(M, part_ml[2 * ((size_t)s * total_rows + row)]);
+  M = warp_max(M);
+  if (lane == 0) red[warp] = M;
+  __syncthreads();
+  M = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+  float L = 0.f;
+  for (int s = tid; s < splits; s += 128) {
+    const float2 ml = *(const float2*)(part_ml + 2 * ((size_t)s * total_rows + row));
+    const float w = ml.x == -INFINITY ? 0.f : expf(ml.x - M);
+    merge_w[s] = w;
+    L = fmaf(w, ml.y, L);
+  }
+  L = warp_sum(L);
+  if (lane == 0) red[4 + warp] = L;
+  __syncthreads();
+  const float inv = 1.0f / ((red[4] + red[5]) + (red[6] + red[7]) + (sink ? expf(sk - M) : 0.f));
+  for (int r = tid * 2; r < rank; r += 256) {
     float a0 = 0.f, a1 = 0.f;
-    for (int s = 0; s < splits; ++s) {
-      const float m = part_ml[2 * ((size_t)s * total_rows + row)];
-      if (m == -INFINITY) continue;
-      const float w = expf(m - M);
-      const float2 v = *(const float2*)(part_o + ((size_t)s * total_rows + row) * rank + r);
-      a0 = fmaf(w, v.x, a0);
-      a1 = fmaf(w, v.y, a1);
+    const float* po = part_o + row * rank + r;
+    const size_t step = (size_t)total_rows * rank;
+    for (int s0 = 0; s0 < splits; s0 += 4) {
+      float2 v[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) v[u] = s0 + u < splits ? *(const float2*)(po + (size_t)(s0 + u) * step) : make_float2(0.f, 0.f);
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const float w = s0 + u < splits ? merge_w[s0 + u] : 0.f;
+        a0 = fmaf(w, v[u].x, a0);
+        a1 = fmaf(w, v[u].y, a1);
+      }
     }
     *(__nv_bfloat162*)(lat + row * rank + r) = __floats2bfloat162_rn(a0 * inv, a1 * inv);
   }
@@ -635,7 +663,7 @@ extern "C" int qv_latent_attention_tc(void* out, int ld_out, const void* q, int 
                                       int dv, int rank, int page, int window, float scale, int splits, void* workspace,
                                       const float* sink, int weight_terms, void* stream) {
   if (T <= 0) return 0;
-  if (rank % 64 || rank > 512 || dr % 16 || dr < 0 || dn % 8 || dn <= 0 || ld_q % 8 || splits < 1 || S > 65535 || splits > 65535 || H > 65535)
+  if (rank % 64 || rank > 512 || dr % 16 || dr < 0 || dn % 8 || dn <= 0 || ld_q % 8 || splits < 1 || S > 65535 || splits > 8192 || H > 65535)
     return QV_ERR_UNSUPPORTED;
   if ((T + 63) / 64 > 65535) return QV_ERR_TOO_LARGE;
   if (weight_terms != 1 && weight_terms != 3) return QV_ERR_UNSUPPORTED;
@@ -674,7 +702,7 @@ extern "C" int qv_latent_attention_tc(void* out, int ld_out, const void* q, int 
 #undef LT_LAUNCH
 #undef LT_LAUNCH_WT
   if (rc) return rc;
-  rc = qv_launch(latent_merge_kernel, dim3((unsigned)rows), dim3(128), 0, st, lat, (const float*)part_o, (const float*)part_ml, rank,
+  rc = qv_launch(latent_merge_kernel, dim3((unsigned)rows), dim3(128), (size_t)splits * sizeof(float), st, lat, (const float*)part_o, (const float*)part_ml, rank,
                  splits, (int)rows, sink, H);
   if (rc) return rc;
   // the heads' value matrices and the gate: per head latent [T, rank] x Wuv_h^T [rank, dv]
